@@ -1,4 +1,5 @@
-"""ctypes binding of libatma_b200.so (the C ABI declared in include/atma_b200.h).
+"""ctypes binding of libatma_b200.so and libatma_decoder.so (the C ABIs declared in include/atma_b200.h and
+include/atma_decoder.h).
 
 There is no fallback: if the library is missing or a call fails, an exception is raised.
 """
@@ -11,6 +12,7 @@ import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libatma_b200.so")
+DECODER_LIB_PATH = os.path.join(_HERE, "libatma_decoder.so")
 
 ATMA_OK, ATMA_ERR_INVALID, ATMA_ERR_CUDA, ATMA_ERR_UNSUPPORTED = 0, -1, -2, -3
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1, torch.float16: 2}
@@ -55,6 +57,32 @@ class PolarDecodeArgs(Structure):
         ("temp_lens", c_void_p), ("skip_merge", c_int),
         ("append_k", c_void_p), ("append_v", c_void_p), ("append_k_stride", c_int64), ("append_v_stride", c_int64),
         ("append_slots", c_void_p),
+    ]
+
+
+class SoftmaxArgs(Structure):
+    """Mirror of atma_softmax_args (include/atma_decoder.h)."""
+    _fields_ = [
+        ("q", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p),
+        ("block_tables", c_void_p), ("bt_stride", c_int64), ("cu_rows", c_void_p), ("start_pos", c_void_p),
+        ("out", c_void_p), ("out_rs", c_int64), ("scratch", c_void_p),
+        ("tile_seq", c_void_p), ("tile_row", c_void_p), ("n_tiles", c_int),
+        ("n_seqs", c_int), ("max_rows", c_int), ("total_rows", c_int),
+        ("H", c_int), ("G", c_int), ("maps", c_int), ("dim", c_int), ("vdim", c_int),
+        ("num_blocks", c_int), ("block_size", c_int), ("max_blocks", c_int), ("n_splits", c_int), ("dtype", c_int),
+        ("scale", c_float), ("lambda_", c_float), ("out_scale", c_float), ("eps", c_float),
+    ]
+
+
+class DeltaArgs(Structure):
+    """Mirror of atma_delta_args (include/atma_decoder.h)."""
+    _fields_ = [
+        ("z", c_void_p), ("z_rs", c_int64), ("conv_q", c_void_p), ("conv_k", c_void_p), ("conv_v", c_void_p),
+        ("A_log", c_void_p), ("dt_bias", c_void_p), ("conv_table", c_void_p), ("conv_ss", c_int64),
+        ("state_table", c_void_p), ("state_ss", c_int64), ("slots", c_void_p), ("cu_rows", c_void_p),
+        ("start_pos", c_void_p), ("row_seq", c_void_p),
+        ("n_seqs", c_int), ("total_rows", c_int), ("H", c_int), ("G", c_int), ("dim", c_int), ("vdim", c_int),
+        ("taps", c_int), ("dtype", c_int), ("unit_eps", c_float), ("q_scale", c_float),
     ]
 
 
@@ -131,33 +159,71 @@ _SIGNATURES = {
                                      c_int, c_float, c_int, c_void_p]),
 }
 
+# libatma_decoder.so (include/atma_decoder.h); the entries it shares with libatma_b200.so have the same signature there
+_DECODER_SIGNATURES = {
+    "atma_decoder_abi_version": (c_int, []),
+    "atma_decoder_device_status": (c_int, [POINTER(c_int)]),
+    "atma_embed_bigram": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int, c_void_p]),
+    "atma_residual_norms": (c_int, [c_void_p] * 7 + [c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "atma_gelu_gate": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
+    "atma_head_norm_silu_gate": (c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_float,
+                                         c_int, c_void_p]),
+    "atma_rotary_store": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p] +
+                          [c_int] * 8 + [c_void_p]),
+    "atma_softmax_prefill": (c_int, [POINTER(SoftmaxArgs), c_void_p]),
+    "atma_softmax_prefill_path": (c_int, [POINTER(SoftmaxArgs)]),
+    "atma_softmax_decode": (c_int, [POINTER(SoftmaxArgs), c_void_p]),
+    "atma_softmax_decode_path": (c_int, [POINTER(SoftmaxArgs)]),
+    "atma_softmax_decode_scratch_floats": (c_int64, [c_int] * 5),
+    "atma_delta_prepare": (c_int, [POINTER(DeltaArgs)] + [c_void_p] * 8),
+    "atma_delta_scan": (c_int, [POINTER(DeltaArgs)] + [c_void_p] * 10),
+    "atma_delta_scan_path": (c_int, [POINTER(DeltaArgs)]),
+    "atma_delta_scan_scratch_bytes": (c_int64, [POINTER(DeltaArgs)]),
+    "atma_delta_step": (c_int, [POINTER(DeltaArgs), c_void_p, c_void_p, c_int64, c_float, c_void_p]),
+}
+_SHARED_SYMBOLS = ("atma_last_error", "atma_decode_linear")
+
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
+DECODER_SYMBOLS = tuple(_DECODER_SIGNATURES)
 
 _lib = None
+_decoder_lib = None
 
 
-def load():
-    """Load the shared library (once).  Raises RuntimeError if it has not been built."""
-    global _lib
-    if _lib is not None:
-        return _lib
-    if not os.path.exists(LIB_PATH):
+def _open(path, target, signatures):
+    if not os.path.exists(path):
         raise RuntimeError(
-            f"{LIB_PATH} is missing: build it with `python -m atma_b200.build` "
+            f"{path} is missing: build it with `python -m atma_b200.build{target}` "
             "(nvcc, sm_100a).  atma_b200 has no CPU or PyTorch fallback.")
-    lib = ctypes.CDLL(LIB_PATH)
-    for name, (res, args) in _SIGNATURES.items():
+    lib = ctypes.CDLL(path)
+    for name, (res, args) in signatures.items():
         fn = getattr(lib, name)          # AttributeError here = header / library mismatch
         fn.restype, fn.argtypes = res, args
-    _lib = lib
     return lib
 
 
-def check(rc):
-    """Turn a C status into the exception the reference API would raise."""
+def load():
+    """Load libatma_b200.so (once).  Raises RuntimeError if it has not been built."""
+    global _lib
+    if _lib is None:
+        _lib = _open(LIB_PATH, "", _SIGNATURES)
+    return _lib
+
+
+def load_decoder():
+    """Load libatma_decoder.so (once).  Raises RuntimeError if it has not been built."""
+    global _decoder_lib
+    if _decoder_lib is None:
+        _decoder_lib = _open(DECODER_LIB_PATH, " decoder", {**_DECODER_SIGNATURES, **{n: _SIGNATURES[n] for n in _SHARED_SYMBOLS}})
+    return _decoder_lib
+
+
+def check(rc, lib=None):
+    """Turn a C status into the exception the reference API would raise.  ``lib``: the library that returned it
+    (each keeps its own message; None = libatma_b200.so)."""
     if rc == ATMA_OK:
         return
-    msg = load().atma_last_error().decode("utf-8", "replace")
+    msg = (load() if lib is None else lib).atma_last_error().decode("utf-8", "replace")
     if rc in (ATMA_ERR_INVALID, ATMA_ERR_UNSUPPORTED):
         raise ValueError(msg)
     raise RuntimeError(msg)

@@ -30,11 +30,11 @@ struct LinArgs {
 };
 
 // One warp: its unit's rows [row0, row0+16) (and, gated, [row0 + N/2, ...)) over k in [k0, k1).
-template <typename T, int NT, bool kGated>
+template <typename T, int NT, int kGated>                  // kGated: 0 plain, 1 up * relu(gate)^2, 2 gelu_tanh(gate) * up
 __global__ void __launch_bounds__(kWarps * 32)
 decode_linear_kernel(const LinArgs a) {
   constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
-  constexpr int kTiles = kGated ? 2 : 1;
+  constexpr int kTiles = kGated != 0 ? 2 : 1;
   __shared__ float part[kWarps][kTiles][NT][4][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -128,7 +128,10 @@ decode_linear_kernel(const LinArgs a) {
       const int feat = row0 + g + (j >= 2 ? 8 : 0);
       if (b >= a.B) continue;
       float v = y[0][j];
-      if constexpr (kGated) {
+      if constexpr (kGated == 2) {
+        const float z = y[0][j];
+        v = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))) * y[1][j];
+      } else if constexpr (kGated == 1) {
         const float p = fmaxf(y[0][j], 0.f);
         float sq = p * p;
         if constexpr (kBf16) sq = round_through<T>(sq);         // eager bf16 materialises relu(x)^2 before the multiply
@@ -166,13 +169,16 @@ extern "C" int atma_decode_linear(const void* x, int64_t x_row_stride, const voi
   const dim3 grid((a.units + upc - 1) / upc), block(kWarps * 32);
   cudaStream_t st = (cudaStream_t)stream;
 #define ATMA_LIN(T, NT, G) decode_linear_kernel<T, NT, G><<<grid, block, 0, st>>>(a)
+#define ATMA_LIN_ANY(T, NT)                                                                  \
+  do {                                                                                       \
+    if (gated == 2) ATMA_LIN(T, NT, 2); else if (gated) ATMA_LIN(T, NT, 1); else ATMA_LIN(T, NT, 0); \
+  } while (0)
   if (dtype == ATMA_BF16) {
-    if (B <= 8) { if (gated) ATMA_LIN(__nv_bfloat16, 1, true); else ATMA_LIN(__nv_bfloat16, 1, false); }
-    else { if (gated) ATMA_LIN(__nv_bfloat16, 2, true); else ATMA_LIN(__nv_bfloat16, 2, false); }
+    if (B <= 8) ATMA_LIN_ANY(__nv_bfloat16, 1); else ATMA_LIN_ANY(__nv_bfloat16, 2);
   } else {
-    if (B <= 8) { if (gated) ATMA_LIN(__half, 1, true); else ATMA_LIN(__half, 1, false); }
-    else { if (gated) ATMA_LIN(__half, 2, true); else ATMA_LIN(__half, 2, false); }
+    if (B <= 8) ATMA_LIN_ANY(__half, 1); else ATMA_LIN_ANY(__half, 2);
   }
+#undef ATMA_LIN_ANY
 #undef ATMA_LIN
   return launch_status("decode_linear");
 }

@@ -1,21 +1,8 @@
 // Bandwidth-bound elementwise kernels of the decode path: squared-ReLU gate, logit
-// soft-cap, KV-cache scatter.  Also hosts the library's error-message plumbing.
+// soft-cap, KV-cache scatter.
 #include "common.cuh"
 
 namespace atma {
-
-char* err_buf() {
-  static thread_local char buf[512] = {0};
-  return buf;
-}
-
-int fail(int code, const char* fmt, ...) {
-  va_list ap;
-  va_start(ap, fmt);
-  vsnprintf(err_buf(), 512, fmt, ap);
-  va_end(ap);
-  return code;
-}
 
 // ---- gate * relu(x)^2 ------------------------------------------------------------------
 // One thread handles VEC consecutive columns of one row (16-byte loads when aligned).
@@ -108,7 +95,6 @@ __global__ void store_kvcache_kernel_bytes2(const char* __restrict__ key, int64_
 
 using namespace atma;
 
-extern "C" const char* atma_last_error(void) { return err_buf(); }
 extern "C" int atma_abi_version(void) { return 1; }
 
 extern "C" int atma_squared_relu_gate(const void* x, int64_t x_stride, const void* gate,

@@ -323,14 +323,19 @@ def decode_linear_supported(x, weight, gated=False):
             weight.is_contiguous() and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0)
 
 
+_GATES = {False: 0, None: 0, True: 1, "squared_relu": 1, "gelu_tanh": 2}
+
+
 @torch.no_grad()
-def decode_linear(x, weight, bias=None, gated=False):
+def decode_linear(x, weight, bias=None, gated=False, out=None, lib=None):
     """x @ weight.T + bias for a decode batch of up to 16 rows, the weights streamed once from HBM
-    (``F.linear`` at these sizes); ``gated``: weight is the MLP's fc projection (2F, K) and the result is
-    second_half * relu(first_half)^2, (rows, F) - the fc GEMM and ``squared_relu_gate`` of
-    inference/models/atma.py:87-97 in one launch.  x (rows, K), weight (N, K) contiguous, 16-bit."""
+    (``F.linear`` at these sizes).  ``gated``: the weight holds two projections (2F, K), first half and second half,
+    and the result is (rows, F): True / "squared_relu" = second * relu(first)^2 - the fc GEMM and
+    ``squared_relu_gate`` of inference/models/atma.py:87-97 in one launch -, "gelu_tanh" = gelu_tanh(first) * second.
+    x (rows, K), weight (N, K) contiguous, 16-bit.  ``out``: where the result goes (contiguous rows, any row stride);
+    ``lib``: the library to call (None = libatma_b200.so; libatma_decoder.so has the same entry)."""
     _lib.require_cuda(x, "decode_linear")
-    lib = _lib.load()
+    lib = _lib.load() if lib is None else lib
     B, K = x.shape
     N = weight.shape[0]
     if weight.shape[1] != K or weight.dtype != x.dtype or not weight.is_contiguous():
@@ -339,7 +344,11 @@ def decode_linear(x, weight, bias=None, gated=False):
         x = x.contiguous()
     if bias is not None:
         bias = bias.to(x.dtype).contiguous()
-    out = torch.empty((B, N // 2 if gated else N), device=x.device, dtype=x.dtype)
+    gate = _GATES[gated]
+    if out is None:
+        out = torch.empty((B, N // 2 if gate else N), device=x.device, dtype=x.dtype)
+    elif out.shape != (B, N // 2 if gate else N) or out.dtype != x.dtype or out.stride(1) != 1:
+        raise ValueError("out must have the result's shape and dtype and contiguous rows")
     _lib.check(lib.atma_decode_linear(_lib.ptr(x), x.stride(0), _lib.ptr(weight), _lib.ptr(bias), _lib.ptr(out), out.stride(0),
-                                      B, N, K, 1 if gated else 0, _lib.dtype_code(x), _lib.stream_ptr()))
+                                      B, N, K, gate, _lib.dtype_code(x), _lib.stream_ptr()), lib)
     return out

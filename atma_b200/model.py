@@ -55,6 +55,29 @@ class ModelState:
 
 
 class AtmaModel:
+    kernel_library = "b200"
+    chunked_prefill = mixed_batches = False       # prompts come whole, in steps of their own
+    graph_decode = True
+
+    @classmethod
+    def from_config(cls, config, tensors, dtype=torch.bfloat16, device="cuda"):
+        """``config``: {"architecture": "Atma", layers, hidden, head_dim, num_kv_heads} and optionally window,
+        gamma_bias, beta_bias, eps; ``tensors``: the reference's state_dict."""
+        kw = {k: config[k] for k in ("layers", "hidden", "head_dim", "num_kv_heads")}
+        kw.update({k: config[k] for k in ("window", "gamma_bias", "beta_bias", "eps") if k in config})
+        return cls(tensors, dtype=dtype, device=device, **kw)
+
+    @torch.no_grad()
+    def forward(self, batch, state):
+        """One engine step (``engine.StepBatch``): fresh prompts, or one token of every decoding sequence."""
+        if batch.prefill is not None:
+            g = batch.prefill
+            h = self.prefill(batch.ids.long(), g.lengths, g.host_slots, state, batch.slot_mapping)
+            return None if batch.logit_rows is None else self.logits(h[batch.logit_rows]).float()
+        g = batch.decode
+        out = self.decode(batch.ids.long(), state, g.slots, batch.slot_mapping.to(torch.int32), g.block_tables, g.start_pos + 1)
+        return None if batch.logit_rows is None else out[batch.logit_rows].float()
+
     def __init__(self, state_dict, *, layers, hidden, head_dim, num_kv_heads, window=None, gamma_bias=3.9, beta_bias=0.0,
                  eps=1e-6, dtype=torch.bfloat16, device="cuda"):
         self.L, self.D, self.dk, self.Hkv = layers, hidden, head_dim, num_kv_heads
@@ -94,7 +117,7 @@ class AtmaModel:
                                   polar={n: sd[P + n] for n in POLAR_NAMES})
 
     # ---- per-sequence device state ---------------------------------------------------------------------
-    def new_state(self, max_seqs, num_blocks, block_size=256):
+    def new_state(self, max_seqs, num_blocks, block_size=256, max_positions=None):
         st = ModelState()
         dev, dt = self.device, self.dtype
         for i in range(self.L):
