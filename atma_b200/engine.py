@@ -152,7 +152,7 @@ class Scheduler:
             self.running.append(self.waiting.popleft())
 
     def schedule(self):
-        """[(sequence, new tokens)]: decoding sequences (1 token) first, then prompt portions."""
+        """[(sequence, new tokens)]: one-token entries first, then longer prompt portions."""
         self._admit()
         decoding = [s for s in self.running if len(s.tokens) - s.done == 1]
         prompts = [s for s in self.running if len(s.tokens) - s.done > 1]
@@ -175,6 +175,8 @@ class Scheduler:
                 continue
             plan.append((s, n))
             budget -= n
+        if self.chunked:
+            plan.sort(key=lambda e: e[1] != 1)              # a portion of one token runs like a decoding sequence
         return plan
 
     def finish(self, seq):
