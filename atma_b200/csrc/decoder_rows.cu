@@ -171,7 +171,10 @@ head_norm_silu_gate_kernel(const T* __restrict__ o, const T* __restrict__ w, con
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       const float gf = to_f32(g.e[e]);
-      r.e[e] = from_f32<T>(to_f32(p.e[e]) * rs * to_f32(wv.e[e]) * (gf / (1.0f + expf(-gf))));
+      float sg;                                          // 16-bit results: the fast exponential and division
+      if constexpr (sizeof(T) == 2) sg = __fdividef(gf, 1.0f + __expf(-gf));
+      else sg = gf / (1.0f + expf(-gf));
+      r.e[e] = from_f32<T>(to_f32(p.e[e]) * rs * to_f32(wv.e[e]) * sg);
     }
     *reinterpret_cast<Pack<T, VEC>*>(outp + c) = r;
   }

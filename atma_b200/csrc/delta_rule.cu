@@ -15,24 +15,31 @@ namespace atma {
 namespace {
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+// for results that are rounded to 16 bits anyway: the fast exponential and division (a few fp32 units in the last place)
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
+  else return silu(x);
+}
 __device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
 
 
-// ---- prepare: one warp = one head of q, k or v (or the gates of all heads) over kRun consecutive rows -------------
-constexpr int kRun = 16;
+// ---- prepare: one warp = one head of q, k or v (or the gates of all heads) over a run of rows -------------
+constexpr int kRunShort = 16, kRunLong = 64;           // rows per warp: short steps need the parallelism
+constexpr int kLongRows = 16384;
 
 template <typename T, int CPL, int KT>
 __global__ void __launch_bounds__(128)
 delta_prepare_kernel(const atma_delta_args a, T* __restrict__ qo, T* __restrict__ ko, T* __restrict__ vo, float* __restrict__ q_inv,
-                     float* __restrict__ k_inv, float* __restrict__ log_decay, float* __restrict__ beta) {
+                     float* __restrict__ k_inv, float* __restrict__ log_decay, float* __restrict__ beta, int run) {
   const int lane = threadIdx.x & 31;
   const int units = 2 * a.G + a.H + 1;
   const int64_t wid = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
   const int u = (int)(wid % units);
-  const int64_t row0 = wid / units * kRun;
+  const int64_t row0 = wid / units * run;
   if (row0 >= a.total_rows) return;
-  const int row1 = (int)min((int64_t)a.total_rows, row0 + kRun);
+  const int row1 = (int)min((int64_t)a.total_rows, row0 + run);
   const T* Z = static_cast<const T*>(a.z);
   const int nq = a.G * a.dim, nv = a.H * a.vdim;
   if (u == units - 1) {                        // gates
@@ -88,60 +95,107 @@ delta_prepare_kernel(const atma_delta_args a, T* __restrict__ qo, T* __restrict_
 #pragma unroll
       for (int i = 0; i < CPL; ++i) w[j][i] = c0 + i < dim ? to_f32(W[(int64_t)(c0 + i) * KT + j]) : 0.f;
   }
-  int seq = -1, first_row = 0, start = 0;
-  int64_t slot = 0;
-  for (int row = (int)row0; row < row1; ++row) {
-    float acc[CPL];
+  // U output rows from their convolution sums
+  auto finish = [&](int row, auto& acc) {
+    constexpr int U = sizeof(acc) / sizeof(acc[0]);
+    float ss[U];
 #pragma unroll
-    for (int i = 0; i < CPL; ++i) acc[i] = 0.f;
-    const int sq = a.row_seq[row];
-    const bool entered = sq != seq;
-    if (entered) { seq = sq; first_row = a.cu_rows[sq]; start = a.start_pos[sq]; slot = a.slots[sq]; }
-    if constexpr (KT > 0) {
-      if (entered) {
+    for (int r = 0; r < U; ++r) {
+      T* op = dst + ((int64_t)(row + r) * heads + head) * dim + c0;
+      Vec o;
+      ss[r] = 0.f;
 #pragma unroll
-        for (int j = 0; j + 1 < KT; ++j) fetch(row, KT - 1 - j, first_row, start, slot, win[j]);
+      for (int i = 0; i < CPL; ++i) {
+        o.e[i] = from_f32<T>(silu_for<T>(acc[r][i]));
+        const float f = c0 + i < dim ? to_f32(o.e[i]) : 0.f;
+        ss[r] = fmaf(f, f, ss[r]);
       }
-      load(Z + (int64_t)row * a.z_rs + zoff + c0, win[KT - 1]);
-#pragma unroll
-      for (int j = 0; j < KT; ++j)
-#pragma unroll
-        for (int i = 0; i < CPL; ++i) acc[i] = fmaf(win[j][i], w[j][i], acc[i]);
-#pragma unroll
-      for (int j = 0; j + 1 < KT; ++j)
-#pragma unroll
-        for (int i = 0; i < CPL; ++i) win[j][i] = win[j + 1][i];
-    } else {
-      for (int j = 0; j < taps; ++j) {
-        float x[CPL];
-        fetch(row, taps - 1 - j, first_row, start, slot, x);
+      if (full && (reinterpret_cast<uintptr_t>(op) & (sizeof(Vec) - 1)) == 0) {
+        *reinterpret_cast<Vec*>(op) = o;
+      } else {
 #pragma unroll
         for (int i = 0; i < CPL; ++i)
-          if (c0 + i < dim) acc[i] = fmaf(x[i], to_f32(W[(int64_t)(c0 + i) * taps + j]), acc[i]);
+          if (c0 + i < dim) op[i] = o.e[i];
       }
     }
-    T* op = dst + ((int64_t)row * heads + head) * dim + c0;
-    float ss = 0.f;
-    Vec o;
-#pragma unroll
-    for (int i = 0; i < CPL; ++i) {
-      o.e[i] = from_f32<T>(silu(acc[i]));
-      const float f = c0 + i < dim ? to_f32(o.e[i]) : 0.f;
-      ss = fmaf(f, f, ss);
-    }
-    if (full && (reinterpret_cast<uintptr_t>(op) & (sizeof(Vec) - 1)) == 0) {
-      *reinterpret_cast<Vec*>(op) = o;
-    } else {
-#pragma unroll
-      for (int i = 0; i < CPL; ++i)
-        if (c0 + i < dim) op[i] = o.e[i];
-    }
     if (part < 2) {
-      ss = warp_sum(ss);
-      if (lane == 0) {
-        const float inv = 1.0f / sqrtf(ss + a.unit_eps);
-        if (part == 0) q_inv[(int64_t)row * a.G + head] = inv * a.q_scale;
-        else k_inv[(int64_t)row * a.G + head] = inv;
+#pragma unroll
+      for (int sft = 16; sft > 0; sft >>= 1)
+#pragma unroll
+        for (int r = 0; r < U; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], sft);
+      float mine = ss[0];
+#pragma unroll
+      for (int r = 1; r < U; ++r) mine = lane == r ? ss[r] : mine;
+      if (lane < U) {
+        const float inv = 1.0f / sqrtf(mine + a.unit_eps);
+        if (part == 0) q_inv[(int64_t)(row + lane) * a.G + head] = inv * a.q_scale;
+        else k_inv[(int64_t)(row + lane) * a.G + head] = inv;
+      }
+    }
+  };
+  for (int row = (int)row0; row < row1;) {
+    const int seq = a.row_seq[row];
+    const int first_row = a.cu_rows[seq], start = a.start_pos[seq], end = min(row1, a.cu_rows[seq + 1]);
+    const int64_t slot = a.slots[seq];
+    if constexpr (KT > 0) {
+#pragma unroll
+      for (int j = 0; j + 1 < KT; ++j) fetch(row, KT - 1 - j, first_row, start, slot, win[j]);
+      constexpr int U = 4;                                      // rows requested together, one group ahead
+      float nxt[U][CPL];
+      auto request = [&](int r0) {
+#pragma unroll
+        for (int r = 0; r < U; ++r) load(Z + (int64_t)min(r0 + r, end - 1) * a.z_rs + zoff + c0, nxt[r]);
+      };
+      if (row + U <= end) request(row);
+      for (; row + U <= end; row += U) {
+        float x[KT - 1 + U][CPL], acc[U][CPL];
+#pragma unroll
+        for (int j = 0; j + 1 < KT; ++j)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) x[j][i] = win[j][i];
+#pragma unroll
+        for (int r = 0; r < U; ++r)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) x[KT - 1 + r][i] = nxt[r][i];
+        if (row + 2 * U <= end) request(row + U);
+#pragma unroll
+        for (int r = 0; r < U; ++r)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) {
+            acc[r][i] = 0.f;
+#pragma unroll
+            for (int j = 0; j < KT; ++j) acc[r][i] = fmaf(x[r + j][i], w[j][i], acc[r][i]);
+          }
+        finish(row, acc);
+#pragma unroll
+        for (int j = 0; j + 1 < KT; ++j)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) win[j][i] = x[U + j][i];
+      }
+      for (; row < end; ++row) {
+        float acc[1][CPL] = {};
+        load(Z + (int64_t)row * a.z_rs + zoff + c0, win[KT - 1]);
+#pragma unroll
+        for (int j = 0; j < KT; ++j)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) acc[0][i] = fmaf(win[j][i], w[j][i], acc[0][i]);
+#pragma unroll
+        for (int j = 0; j + 1 < KT; ++j)
+#pragma unroll
+          for (int i = 0; i < CPL; ++i) win[j][i] = win[j + 1][i];
+        finish(row, acc);
+      }
+    } else {
+      for (; row < end; ++row) {
+        float acc[1][CPL] = {};
+        for (int j = 0; j < taps; ++j) {
+          float x[CPL];
+          fetch(row, taps - 1 - j, first_row, start, slot, x);
+#pragma unroll
+          for (int i = 0; i < CPL; ++i)
+            if (c0 + i < dim) acc[0][i] = fmaf(x[i], to_f32(W[(int64_t)(c0 + i) * taps + j]), acc[0][i]);
+        }
+        finish(row, acc);
       }
     }
   }
@@ -257,7 +311,7 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
   float* s_k = s_q + K;                         // [K]
   float* s_v = s_k + K;                         // [V]
   float* s_o = s_v + V;                         // [V]
-  __shared__ float s_red[kStepWarps][32 * VEC];
+  __shared__ __align__(16) float s_red[kStepWarps][32 * VEC];
   __shared__ float s_sum[3][kStepWarps];
   const int b = blockIdx.y, h = blockIdx.x;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -291,6 +345,7 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
   const int nq = a.G * K, ctot = 2 * nq + a.H * V, taps = a.taps;
   const T* zr = static_cast<const T*>(a.z) + b * a.z_rs;
   T* table = static_cast<T*>(a.conv_table) + slot * a.conv_ss;
+  const int ring = pos % taps;
   float qs = 0.f, ks = 0.f;
   for (int i = tid; i < 2 * K + V; i += kStepWarps * 32) {
     const int part = i < K ? 0 : (i < 2 * K ? 1 : 2);
@@ -301,9 +356,9 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
     const T cur = zr[zc];
     float acc = to_f32(cur) * to_f32(w[taps - 1]);
     for (int j = 1; j < taps; ++j)
-      if (pos - j >= 0) acc = fmaf(to_f32(table[(int64_t)((pos - j) % taps) * ctot + zc]), to_f32(w[taps - 1 - j]), acc);
-    if (part == 2 || h % rep == 0) table[(int64_t)(pos % taps) * ctot + zc] = cur;
-    const float y = round_through<T>(silu(acc));
+      if (pos - j >= 0) acc = fmaf(to_f32(table[(int64_t)(ring - j + (ring < j ? taps : 0)) * ctot + zc]), to_f32(w[taps - 1 - j]), acc);
+    if (part == 2 || h % rep == 0) table[(int64_t)ring * ctot + zc] = cur;
+    const float y = round_through<T>(silu_for<T>(acc));
     if (part == 0) { s_q[c] = y; qs = fmaf(y, y, qs); }
     else if (part == 1) { s_k[c] = y; ks = fmaf(y, y, ks); }
     else s_v[c] = y;
@@ -323,7 +378,7 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
   for (int cb = 0; cb < cblocks; ++cb) {
     if (cb > 0) load_state(cb);
     const int c = cb * 32 * VEC + lane * VEC;
-    float p[VEC] = {};
+    alignas(16) float p[VEC] = {};
 #pragma unroll
     for (int i = 0; i < RPW; ++i) {
       const int r = warp + kStepWarps * i;
@@ -332,17 +387,18 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
       for (int e = 0; e < VEC; ++e) { S[i].e[e] *= gm; p[e] = fmaf(kn, S[i].e[e], p[e]); }
     }
     __syncthreads();                            // s_red is free again
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) s_red[warp][lane * VEC + e] = p[e];
+    *reinterpret_cast<FV*>(&s_red[warp][lane * VEC]) = *reinterpret_cast<const FV*>(p);
     __syncthreads();
-    float u[VEC], rd[VEC] = {};
+    alignas(16) float rd[VEC] = {};
+    float u[VEC] = {};
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) {
-      float t = 0.f;
+    for (int w = 0; w < kStepWarps; ++w) {
+      const FV t = *reinterpret_cast<const FV*>(&s_red[w][lane * VEC]);
 #pragma unroll
-      for (int w = 0; w < kStepWarps; ++w) t += s_red[w][lane * VEC + e];
-      u[e] = c + e < V ? bt * (s_v[c + e] - t) : 0.f;
+      for (int e = 0; e < VEC; ++e) u[e] += t.e[e];
     }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u[e] = c + e < V ? bt * (s_v[c + e] - u[e]) : 0.f;
 #pragma unroll
     for (int i = 0; i < RPW; ++i) {
       const int r = warp + kStepWarps * i;
@@ -354,8 +410,7 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
       }
     }
     __syncthreads();
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) s_red[warp][lane * VEC + e] = rd[e];
+    *reinterpret_cast<FV*>(&s_red[warp][lane * VEC]) = *reinterpret_cast<const FV*>(rd);
     __syncthreads();
     if (tid < 32 * VEC) {
       const int cc = cb * 32 * VEC + tid;
@@ -389,9 +444,10 @@ int check(const atma_delta_args* a, const char* what) {
 
 template <typename T, int CPL>
 int launch_prepare(const atma_delta_args& a, void* q, void* k, void* v, float* qi, float* ki, float* ld, float* bt, cudaStream_t st) {
-  const int64_t warps = (int64_t)((a.total_rows + kRun - 1) / kRun) * (2 * a.G + a.H + 1);
+  const int run = a.total_rows >= kLongRows ? kRunLong : kRunShort;
+  const int64_t warps = (int64_t)((a.total_rows + run - 1) / run) * (2 * a.G + a.H + 1);
   const unsigned grid = (unsigned)((warps + 3) / 4);
-#define ATMA_PREP(KT) delta_prepare_kernel<T, CPL, KT><<<grid, 128, 0, st>>>(a, (T*)q, (T*)k, (T*)v, qi, ki, ld, bt)
+#define ATMA_PREP(KT) delta_prepare_kernel<T, CPL, KT><<<grid, 128, 0, st>>>(a, (T*)q, (T*)k, (T*)v, qi, ki, ld, bt, run)
   switch (a.taps) {
     case 2: ATMA_PREP(2); break;
     case 3: ATMA_PREP(3); break;

@@ -34,7 +34,7 @@ namespace {
 __device__ int g_delta_status = 0;
 
 constexpr int kC = 64, kD = 128;
-constexpr int kRecBytes = 4 * kC * kC * 2;          // M1 hi, M1 lo, M2 hi, M2 lo: [64 p][64 s] 16-bit each
+constexpr int kRecBytes = 4 * kC * kC * 2;          // M1 hi, M2 hi, M1 lo, M2 lo: [64 p][64 s] 16-bit each
 constexpr int kScal = 256;                          // floats per record: a k_inv [64] | a q_inv [64] | (a_C/a) k_inv [64] | a_C
 constexpr int kThreads = 320;
 
@@ -346,9 +346,9 @@ delta_factors_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
             split2(x, y, hi[e], lo[e]);
           }
           *reinterpret_cast<uint4*>(r1 + c4 * 16) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(r1 + 8192 + c4 * 16) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          *reinterpret_cast<uint4*>(r1 + 16384 + c4 * 16) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           if (above) {
-            *reinterpret_cast<uint4*>(r1 + 16384 + c4 * 16) = make_uint4(0u, 0u, 0u, 0u);
+            *reinterpret_cast<uint4*>(r1 + 8192 + c4 * 16) = make_uint4(0u, 0u, 0u, 0u);
             *reinterpret_cast<uint4*>(r1 + 24576 + c4 * 16) = make_uint4(0u, 0u, 0u, 0u);
           }
         }
@@ -370,7 +370,7 @@ delta_factors_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
             block_mma(acc, Rf + (64 * cc + 16 * bi) * kLd + 16 * l, Tf + (64 * cc + 16 * l) * kLd + 16 * bj, lane);
           if (rc >= 0) {
             const int g = lane >> 2, t2 = 2 * (lane & 3);
-            uint8_t* r2 = p.recs + rc * (int64_t)kRecBytes + 16384;
+            uint8_t* r2 = p.recs + rc * (int64_t)kRecBytes + 8192;
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
               const int s = 16 * bj + 8 * nt + t2;
@@ -381,7 +381,7 @@ delta_factors_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
                 split2(acc[nt][2 * e] * b0, acc[nt][2 * e + 1] * b1, hi, lo);
                 uint8_t* dst = r2 + (16 * bi + g + 8 * e) * 128 + s * 2;
                 *reinterpret_cast<uint32_t*>(dst) = hi;
-                *reinterpret_cast<uint32_t*>(dst + 8192) = lo;
+                *reinterpret_cast<uint32_t*>(dst + 16384) = lo;
               }
             }
           }
@@ -400,13 +400,15 @@ delta_factors_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
 
 // ======================================= recurrence =======================================================================
 constexpr int kStages = 2;
-constexpr int kOffRK = 0, kOffRQ = 16384, kOffRV = 32768, kOffRM = 49152, kOffRS = 81920, kStageBytes = 82944;   // ... M1, M2 | scalars
+// a stage: [K rows; Q rows] as two boxes of 64 channels x 128 rows | V, two boxes of 64 channels x 64 rows | [M1; M2] rounded,
+// [M1; M2] remainders | scalars
+constexpr int kOffKQ = 0, kOffRV = 32768, kOffRM = 49152, kOffRS = 81920, kStageBytes = 82944;
 constexpr int kRecurSmem = kStages * kStageBytes + 1024;
-constexpr uint32_t kColS = 0, kColP = 128, kColD = 192, kColR = 320, kColU = 384, kColQ = 448;
+constexpr uint32_t kColS = 0, kColP = 128, kColQ = 192, kColD = 128, kColX = 256, kColX2 = 320, kColR = 384, kColU = 448;
 
 struct RecurBarriers {
   uint64_t in_full[kStages], m_full[kStages], empty[kStages];
-  uint64_t s_ready, p_full, r_ready, u_full, us_ready, s_done, o_done, o_free;
+  uint64_t s_ready, pq_full, r_ready, uo_full, us_ready, s_done;
 };
 
 __global__ void __launch_bounds__(kThreads, 1)
@@ -429,8 +431,8 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 
   if (tid == 0) {
     for (int i = 0; i < kStages; ++i) { mbar_init(&bar.in_full[i], 1); mbar_init(&bar.m_full[i], 1); mbar_init(&bar.empty[i], 9); }
-    mbar_init(&bar.s_ready, 8); mbar_init(&bar.r_ready, 8); mbar_init(&bar.us_ready, 8); mbar_init(&bar.o_free, 8);
-    mbar_init(&bar.p_full, 1); mbar_init(&bar.u_full, 1); mbar_init(&bar.s_done, 1); mbar_init(&bar.o_done, 1);
+    mbar_init(&bar.s_ready, 8); mbar_init(&bar.r_ready, 8); mbar_init(&bar.us_ready, 8);
+    mbar_init(&bar.pq_full, 1); mbar_init(&bar.uo_full, 1); mbar_init(&bar.s_done, 1);
     s_abort = 0;
     fence_barrier_init();
   }
@@ -454,8 +456,8 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         mbar_arrive_expect_tx(&bar.in_full[s], 3 * 16384 + 1024);
 #pragma unroll
         for (int cb = 0; cb < 2; ++cb) {
-          tma_load_4d(st + kOffRK + cb * 8192, &tmap_k, &bar.in_full[s], cb * 64, g, t0, 0);
-          tma_load_4d(st + kOffRQ + cb * 8192, &tmap_q, &bar.in_full[s], cb * 64, g, t0, 0);
+          tma_load_4d(st + kOffKQ + cb * 16384, &tmap_k, &bar.in_full[s], cb * 64, g, t0, 0);
+          tma_load_4d(st + kOffKQ + cb * 16384 + 8192, &tmap_q, &bar.in_full[s], cb * 64, g, t0, 0);
           tma_load_4d(st + kOffRV + cb * 8192, &tmap_v, &bar.in_full[s], cb * 64, hv, t0, 0);
         }
         bulk_load(st + kOffRS, p.scal + rec * kScal, kScal * 4, &bar.in_full[s]);
@@ -468,17 +470,17 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   } else if (warp == 1) {
     // ---- MMA issuer --------------------------------------------------------------------------------------------
     if (lane == 0) {
-      constexpr uint32_t idesc_n64 = make_idesc(128, 64, 1, 0, 0);
-      constexpr uint32_t idesc_ds = make_idesc(128, 128, 1, 0, 1);
+      constexpr uint32_t idesc_k = make_idesc(128, 128, 1, 0, 0);      // B rows as they lie: [K; Q] or [M1; M2]
+      constexpr uint32_t idesc_ds = make_idesc(128, 128, 1, 0, 1);     // B = K [s][k], MN-major
       const uint64_t hi_k = (uint64_t(1024 >> 4) << 32) | (uint64_t(1) << 46) | (uint64_t(2) << 61) | (uint64_t(16 >> 4) << 16);
-      const uint64_t hi_mn = (uint64_t(1024 >> 4) << 32) | (uint64_t(1) << 46) | (uint64_t(2) << 61) | (uint64_t(8192 >> 4) << 16);
+      const uint64_t hi_mn = (uint64_t(1024 >> 4) << 32) | (uint64_t(1) << 46) | (uint64_t(2) << 61) | (uint64_t(16384 >> 4) << 16);
       bool ok = true;
       for (int i = 0; i < n_chunks && ok; ++i) {
         const int s = i % kStages;
         const uint32_t ph = (uint32_t)(i / kStages) & 1u, pi = (uint32_t)i & 1u;
         const uint32_t st = smem_u32(smem + s * kStageBytes);
-        const uint64_t kd = hi_k | uint64_t(((st + kOffRK) >> 4) & 0x3FFFu), qd = hi_k | uint64_t(((st + kOffRQ) >> 4) & 0x3FFFu);
-        const uint64_t kmn = hi_mn | uint64_t(((st + kOffRK) >> 4) & 0x3FFFu), md = hi_k | uint64_t(((st + kOffRM) >> 4) & 0x3FFFu);
+        const uint64_t kq = hi_k | uint64_t(((st + kOffKQ) >> 4) & 0x3FFFu), kmn = hi_mn | uint64_t(((st + kOffKQ) >> 4) & 0x3FFFu);
+        const uint64_t md = hi_k | uint64_t(((st + kOffRM) >> 4) & 0x3FFFu);
         ok = mbar_wait(&bar.s_ready, pi, abort_flag) && mbar_wait(&bar.in_full[s], ph, abort_flag);
         if (!ok) break;
         tc_fence_after();
@@ -486,29 +488,20 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         for (int term = 0; term < 2; ++term)
 #pragma unroll
           for (int kk = 0; kk < 8; ++kk)
-            mma_ts(tbase + kColP, tbase + kColS + term * 64 + kk * 8, kd + uint64_t(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), idesc_n64,
+            mma_ts(tbase + kColP, tbase + kColS + term * 64 + kk * 8, kq + uint64_t(((kk >> 2) * 16384 + (kk & 3) * 32) >> 4), idesc_k,
                    (term > 0 || kk > 0) ? 1u : 0u);
-        tc_commit(&bar.p_full);
-        if (i > 0) ok = mbar_wait(&bar.o_free, (uint32_t)(i - 1) & 1u, abort_flag);
-        if (!ok) break;
-        tc_fence_after();
-#pragma unroll
-        for (int kk = 0; kk < 8; ++kk)
-          mma_ts(tbase + kColQ, tbase + kColS + kk * 8, qd + uint64_t(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), idesc_n64, kk > 0);
+        tc_commit(&bar.pq_full);
         ok = mbar_wait(&bar.r_ready, pi, abort_flag) && mbar_wait(&bar.m_full[s], ph, abort_flag);
         if (!ok) break;
         tc_fence_after();
-        // U^T = R^T M1^T: (hi, hi), (lo, hi), (hi, lo)
+        // (rounded, rounded), (remainder, rounded), (rounded, remainder)
 #pragma unroll
         for (int term = 0; term < 3; ++term)
 #pragma unroll
           for (int kk = 0; kk < 4; ++kk)
-            mma_ts(tbase + kColP, tbase + kColR + (term == 1 ? 32 : 0) + kk * 8, md + uint64_t(((term == 2 ? 8192 : 0) + kk * 32) >> 4), idesc_n64,
+            mma_ts(tbase + kColX, tbase + kColR + (term == 1 ? 32 : 0) + kk * 8, md + uint64_t(((term == 2 ? 16384 : 0) + kk * 32) >> 4), idesc_k,
                    (term > 0 || kk > 0) ? 1u : 0u);
-        tc_commit(&bar.u_full);
-#pragma unroll
-        for (int kk = 0; kk < 8; ++kk)
-          mma_ts(tbase + kColQ, tbase + kColS + 64 + kk * 8, qd + uint64_t(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), idesc_n64, 1u);
+        tc_commit(&bar.uo_full);
         ok = mbar_wait(&bar.us_ready, pi, abort_flag);
         if (!ok) break;
         tc_fence_after();
@@ -518,14 +511,6 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           for (int kk = 0; kk < 4; ++kk)
             mma_ts(tbase + kColD, tbase + kColU + term * 32 + kk * 8, kmn + uint64_t((kk * 2048) >> 4), idesc_ds, (term > 0 || kk > 0) ? 1u : 0u);
         tc_commit(&bar.s_done);
-        // R^T M2^T, over the 16-bit U terms that the products above have read
-#pragma unroll
-        for (int term = 0; term < 3; ++term)
-#pragma unroll
-          for (int kk = 0; kk < 4; ++kk)
-            mma_ts(tbase + kColU, tbase + kColR + (term == 1 ? 32 : 0) + kk * 8, md + uint64_t((16384 + (term == 2 ? 8192 : 0) + kk * 32) >> 4),
-                   idesc_n64, (term > 0 || kk > 0) ? 1u : 0u);
-        tc_commit(&bar.o_done);
         tc_commit(&bar.empty[s]);
       }
     }
@@ -538,22 +523,22 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const int vcol = (hv % vblocks) * kD + v;
     float* plane = p.state + slot * p.state_ss + ((int64_t)h * kD + 64 * half) * p.vdim + vcol;   // element (k = 64 half + j, v)
     const bool fresh = p.start_pos[b] == 0;
-    const int64_t orow = (int64_t)p.H * p.vdim;
     float S[64];
     {
       const float* src = plane;
+      int64_t step = p.vdim;
+      asm volatile("" : "+l"(step));
 #pragma unroll
-      for (int j = 0; j < 64; ++j) { S[j] = fresh ? 0.f : *src; src += p.vdim; }
+      for (int j = 0; j < 64; ++j) { S[j] = fresh ? 0.f : *src; src += step; }
     }
+    float gC = 0.f;                                    // decay over the chunk before
     bool ok = true;
     for (int i = 0; i <= n_chunks; ++i) {
       if (i > 0) {                                     // the state after chunk i - 1
-        const int s = (i - 1) % kStages;
         ok = mbar_wait(&bar.s_done, (uint32_t)(i - 1) & 1u, abort_flag);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
-        const float gC = reinterpret_cast<const float*>(smem + s * kStageBytes + kOffRS)[192];
 #pragma unroll
         for (int q = 0; q < 2; ++q) {
           uint32_t d[32];
@@ -562,70 +547,34 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           for (int j = 0; j < 32; ++j) S[32 * q + j] = fmaf(gC, S[32 * q + j], __uint_as_float(d[j]));
         }
       }
-      if (i < n_chunks) {                              // S^T as two 16-bit terms
-#pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          uint32_t hi[16], lo[16];
-#pragma unroll
-          for (int j = 0; j < 16; ++j) split2(S[32 * q + 2 * j], S[32 * q + 2 * j + 1], hi[j], lo[j]);
-          tmem_st16(lane_base + kColS + 32 * half + 16 * q, hi);
-          tmem_st16(lane_base + kColS + 64 + 32 * half + 16 * q, lo);
-        }
-        tmem_st_wait();
-        tc_fence_before();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&bar.s_ready);
-      } else {
-#pragma unroll
-        for (int j = 0; j < 64; ++j) { *plane = S[j]; plane += p.vdim; }
-      }
-      if (i > 0) {                                     // O of chunk i - 1: rows 32 half .. + 31
-        const int c = i - 1, s = c % kStages;
-        ok = mbar_wait(&bar.o_done, (uint32_t)c & 1u, abort_flag);
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
-        tc_fence_after();
-        uint32_t a[32], r[32];
-        tmem_ld32_nowait(lane_base + kColQ + 32 * half, a);
-        tmem_ld32_nowait(lane_base + kColU + 32 * half, r);
-        tmem_ld_wait();
-        const float* eq = reinterpret_cast<const float*>(smem + s * kStageBytes + kOffRS) + 64 + 32 * half;
-        const int t0 = row_begin + c * kC + 32 * half;
-        const int n_ok = min(32, row_end - t0);
-        uint32_t w[16];                                 // two rows each
-#pragma unroll
-        for (int j = 0; j < 32; j += 4) {
-          const float4 e = *reinterpret_cast<const float4*>(eq + j);
-#pragma unroll
-          for (int q = 0; q < 4; ++q) { reg_fence(a[j + q]); reg_fence(r[j + q]); }
-          w[j >> 1] = pack_bf16(fmaf(e.x, __uint_as_float(a[j]), __uint_as_float(r[j])), fmaf(e.y, __uint_as_float(a[j + 1]), __uint_as_float(r[j + 1])));
-          w[(j >> 1) + 1] = pack_bf16(fmaf(e.z, __uint_as_float(a[j + 2]), __uint_as_float(r[j + 2])),
-                                      fmaf(e.w, __uint_as_float(a[j + 3]), __uint_as_float(r[j + 3])));
-        }
-        tc_fence_before();
-        __syncwarp();
-        if (lane == 0) { mbar_arrive(&bar.o_free); mbar_arrive(&bar.empty[s]); }
-        uint16_t* oc = static_cast<uint16_t*>(p.o) + ((int64_t)t0 * p.H + h) * p.vdim + vcol;
-#pragma unroll
-        for (int j = 0; j < 32; ++j) {
-          if (j < n_ok) *oc = (uint16_t)(w[j >> 1] >> (16 * (j & 1)));
-          oc += orow;
-        }
-      }
       if (i == n_chunks) break;
+      // ---- S^T as two 16-bit terms (the dS columns have been read: the next products may overwrite them) ----
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        uint32_t hi[16], lo[16];
+#pragma unroll
+        for (int j = 0; j < 16; ++j) split2(S[32 * q + 2 * j], S[32 * q + 2 * j + 1], hi[j], lo[j]);
+        tmem_st16(lane_base + kColS + 32 * half + 16 * q, hi);
+        tmem_st16(lane_base + kColS + 64 + 32 * half + 16 * q, lo);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bar.s_ready);
+
       const int s = i % kStages;
       const uint8_t* st = smem + s * kStageBytes;
       const float* sc = reinterpret_cast<const float*>(st + kOffRS);
       // ---- R^T = V^T - (a k_inv) P: this thread's value channel, rows 32 half .. + 31 ----
-      ok = mbar_wait(&bar.in_full[s], (uint32_t)(i / kStages) & 1u, abort_flag) && mbar_wait(&bar.p_full, (uint32_t)i & 1u, abort_flag);
+      ok = mbar_wait(&bar.in_full[s], (uint32_t)(i / kStages) & 1u, abort_flag) && mbar_wait(&bar.pq_full, (uint32_t)i & 1u, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
       {
-        uint32_t pr[32], hi[16], lo[16];
-        tmem_ld32(lane_base + kColP + 32 * half, pr);
         const uint8_t* vb = st + kOffRV + (v >> 6) * 8192 + (v & 7) * 2;
         const int ch = (v & 63) >> 3;
+        uint32_t pr[32], hi[16], lo[16];
+        tmem_ld32(lane_base + kColP + 32 * half, pr);
 #pragma unroll
         for (int j = 0; j < 32; j += 4) {
           const float4 ek = *reinterpret_cast<const float4*>(sc + 32 * half + j);
@@ -647,19 +596,26 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         __syncwarp();
         if (lane == 0) mbar_arrive(&bar.r_ready);
       }
-      // ---- U^T scaled by (a_C / a) k_inv ----
-      ok = mbar_wait(&bar.u_full, (uint32_t)i & 1u, abort_flag);
+      // ---- U^T scaled by (a_C / a) k_inv; S^T Q^T leaves the columns that dS will take ----
+      ok = mbar_wait(&bar.uo_full, (uint32_t)i & 1u, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
+      uint32_t sq[32];
+      tmem_ld32(lane_base + kColQ + 32 * half, sq);
       {
-        uint32_t u[32], hi[16], lo[16];
-        tmem_ld32(lane_base + kColP + 32 * half, u);
+        uint32_t hi[16], lo[16];
 #pragma unroll
-        for (int j = 0; j < 32; j += 4) {
-          const float4 ed = *reinterpret_cast<const float4*>(sc + 128 + 32 * half + j);
-          split2(__uint_as_float(u[j]) * ed.x, __uint_as_float(u[j + 1]) * ed.y, hi[j >> 1], lo[j >> 1]);
-          split2(__uint_as_float(u[j + 2]) * ed.z, __uint_as_float(u[j + 3]) * ed.w, hi[(j >> 1) + 1], lo[(j >> 1) + 1]);
+        for (int q = 0; q < 2; ++q) {
+          uint32_t u[16];
+          tmem_ld16(lane_base + kColX + 32 * half + 16 * q, u);
+#pragma unroll
+          for (int j = 0; j < 16; j += 4) {
+            const float4 ed = *reinterpret_cast<const float4*>(sc + 128 + 32 * half + 16 * q + j);
+            const int w = (16 * q + j) >> 1;
+            split2(__uint_as_float(u[j]) * ed.x, __uint_as_float(u[j + 1]) * ed.y, hi[w], lo[w]);
+            split2(__uint_as_float(u[j + 2]) * ed.z, __uint_as_float(u[j + 3]) * ed.w, hi[w + 1], lo[w + 1]);
+          }
         }
         tmem_st16(lane_base + kColU + 16 * half, hi);
         tmem_st16(lane_base + kColU + 32 + 16 * half, lo);
@@ -668,6 +624,45 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         __syncwarp();
         if (lane == 0) mbar_arrive(&bar.us_ready);
       }
+      // ---- O = (a q_inv) S Q + R M2, under the last product ----
+      {
+        gC = sc[192];
+        const int t0 = row_begin + i * kC + 32 * half;
+        const int n_ok = min(32, row_end - t0);
+        uint16_t* oc = static_cast<uint16_t*>(p.o) + ((int64_t)t0 * p.H + h) * p.vdim + vcol;
+        int64_t orow = (int64_t)p.H * p.vdim;
+        asm volatile("" : "+l"(orow));                  // not a loop invariant: its 31 multiples would be kept in registers
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          uint32_t r[16];
+          tmem_ld16(lane_base + kColX2 + 32 * half + 16 * q, r);
+#pragma unroll
+          for (int j = 0; j < 16; j += 4) {
+            const float4 e = *reinterpret_cast<const float4*>(sc + 64 + 32 * half + 16 * q + j);
+            const uint32_t w0 = pack_bf16(fmaf(e.x, __uint_as_float(sq[16 * q + j]), __uint_as_float(r[j])),
+                                          fmaf(e.y, __uint_as_float(sq[16 * q + j + 1]), __uint_as_float(r[j + 1])));
+            const uint32_t w1 = pack_bf16(fmaf(e.z, __uint_as_float(sq[16 * q + j + 2]), __uint_as_float(r[j + 2])),
+                                          fmaf(e.w, __uint_as_float(sq[16 * q + j + 3]), __uint_as_float(r[j + 3])));
+            if (16 * q + j < n_ok) *oc = (uint16_t)(w0 & 0xffffu);
+            oc += orow;
+            if (16 * q + j + 1 < n_ok) *oc = (uint16_t)(w0 >> 16);
+            oc += orow;
+            if (16 * q + j + 2 < n_ok) *oc = (uint16_t)(w1 & 0xffffu);
+            oc += orow;
+            if (16 * q + j + 3 < n_ok) *oc = (uint16_t)(w1 >> 16);
+            oc += orow;
+          }
+        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&bar.empty[s]);
+      }
+    }
+    if (ok) {
+      int64_t step = p.vdim;
+      asm volatile("" : "+l"(step));                    // opaque, like orow
+#pragma unroll
+      for (int j = 0; j < 64; ++j) { *plane = S[j]; plane += step; }
     }
   }
   tc_fence_before();

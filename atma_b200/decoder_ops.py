@@ -108,10 +108,11 @@ def softmax_prefill(q, k_cache, v_cache, group, out, *, scale, lam=0.0, out_scal
     return out
 
 
-def decode_key_ranges(n_seqs, kv_heads, max_keys):
-    """Key ranges per sequence and key/value head: two resident waves of CTAs, at least 128 keys per range."""
-    want = -(-2 * 148 * 2 // max(1, n_seqs * kv_heads))
-    return max(1, min(want, max_keys // 128, 64))
+def decode_key_ranges(n_seqs, heads, kv_heads, maps, max_keys):
+    """Key ranges per sequence and group of query heads for ``softmax_decode`` (launch-time shapes only)."""
+    from .polar import decode_num_splits
+    per_cta = 8 // maps
+    return decode_num_splits(n_seqs, kv_heads * -(-(heads // kv_heads) // per_cta), max_keys, min_keys=256)
 
 
 def softmax_decode(q, k_cache, v_cache, group, out, *, scale, lam=0.0, out_scale=1.0, eps=0.0, n_splits=None):
@@ -121,7 +122,7 @@ def softmax_decode(q, k_cache, v_cache, group, out, *, scale, lam=0.0, out_scale
     a = _softmax_args(q, k_cache, v_cache, group, out, scale, lam, out_scale, eps)
     scratch = None
     if lib.atma_softmax_decode_path(ctypes.byref(a)):
-        a.n_splits = n_splits or decode_key_ranges(a.n_seqs, a.G, a.max_blocks * a.block_size)
+        a.n_splits = n_splits or decode_key_ranges(a.n_seqs, a.H, a.G, a.maps, a.max_blocks * a.block_size)
         scratch = torch.empty(int(lib.atma_softmax_decode_scratch_floats(a.n_seqs, a.H, a.maps, a.vdim, a.n_splits)),
                               device=q.device, dtype=torch.float32)
         a.scratch = scratch.data_ptr()
@@ -157,27 +158,44 @@ class DeltaWeights:
         return a
 
 
+class DeltaParts:
+    """The two halves of ``delta_prefill`` on buffers of their own: ``prepare`` (convolutions, unit-norm factors, gates,
+    convolution state) and ``scan`` (the recurrence; its result is ``o`` (rows, heads, vdim))."""
+
+    def __init__(self, z, weights, conv_table, state_table, group):
+        _lib.require_cuda(z, "delta_prefill")
+        w, n, dev = weights, z.shape[0], z.device
+        self.lib, self.keep = _lib.load_decoder(), (z, weights, conv_table, state_table, group)
+        self.args = w.args(z, conv_table, state_table, group)
+        self.q = torch.empty((n, w.kv_heads, w.dim), device=dev, dtype=z.dtype)
+        self.k = torch.empty_like(self.q)
+        self.v = torch.empty((n, w.heads, w.vdim), device=dev, dtype=z.dtype)
+        self.inv = torch.empty((2, n, w.kv_heads), device=dev, dtype=torch.float32)
+        self.gates = torch.empty((2, n, w.heads), device=dev, dtype=torch.float32)
+        self.o = torch.empty_like(self.v)
+        nbytes = int(self.lib.atma_delta_scan_scratch_bytes(ctypes.byref(self.args)))
+        self.scratch = torch.empty(nbytes, device=dev, dtype=torch.uint8) if nbytes > 0 else None
+
+    def _factors(self):
+        return _ptr(self.inv[0]), _ptr(self.inv[1]), _ptr(self.gates[0]), _ptr(self.gates[1])
+
+    def prepare(self):
+        _check(self.lib.atma_delta_prepare(ctypes.byref(self.args), _ptr(self.q), _ptr(self.k), _ptr(self.v), *self._factors(), _lib.stream_ptr()))
+
+    def scan(self):
+        _check(self.lib.atma_delta_scan(ctypes.byref(self.args), _ptr(self.q), _ptr(self.k), _ptr(self.v), *self._factors(), _ptr(self.o),
+                                        _ptr(self.scratch), _lib.stream_ptr()))
+
+
 def delta_prefill(z, weights, conv_table, state_table, group, out, eps):
     """The delta mixer between its input and output projections for a group's rows: z rows [q | k | v | gate | a | b],
     conv_table (slots, taps, channels), state_table (slots, heads, dim, vdim) fp32, both updated in place; out
     (rows, heads*vdim)."""
-    _lib.require_cuda(z, "delta_prefill")
-    lib, w, n, dev = _lib.load_decoder(), weights, z.shape[0], z.device
-    a = w.args(z, conv_table, state_table, group)
-    q = torch.empty((n, w.kv_heads, w.dim), device=dev, dtype=z.dtype)
-    k = torch.empty_like(q)
-    v = torch.empty((n, w.heads, w.vdim), device=dev, dtype=z.dtype)
-    inv = torch.empty((2, n, w.kv_heads), device=dev, dtype=torch.float32)
-    gates = torch.empty((2, n, w.heads), device=dev, dtype=torch.float32)
-    _check(lib.atma_delta_prepare(ctypes.byref(a), _ptr(q), _ptr(k), _ptr(v), _ptr(inv[0]), _ptr(inv[1]), _ptr(gates[0]), _ptr(gates[1]),
-                                  _lib.stream_ptr()))
-    o = torch.empty_like(v)
-    nbytes = int(lib.atma_delta_scan_scratch_bytes(ctypes.byref(a)))
-    scratch = torch.empty(nbytes, device=dev, dtype=torch.uint8) if nbytes > 0 else None
-    _check(lib.atma_delta_scan(ctypes.byref(a), _ptr(q), _ptr(k), _ptr(v), _ptr(inv[0]), _ptr(inv[1]), _ptr(gates[0]), _ptr(gates[1]),
-                               _ptr(o), _ptr(scratch), _lib.stream_ptr()))
-    g0 = w.channels
-    return head_norm_silu_gate(o, w.norm, z[:, g0:g0 + w.heads * w.vdim], out, eps)
+    parts = DeltaParts(z, weights, conv_table, state_table, group)
+    parts.prepare()
+    parts.scan()
+    g0 = weights.channels
+    return head_norm_silu_gate(parts.o, weights.norm, z[:, g0:g0 + weights.heads * weights.vdim], out, eps)
 
 
 def delta_step(z, weights, conv_table, state_table, group, out, eps):

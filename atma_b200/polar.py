@@ -196,15 +196,15 @@ def _sm_count(device=None):
     return _sm_counts[idx]
 
 
-def decode_num_splits(B, Hkv, max_context, sm_count=None, ctas_per_sm=2):
+def decode_num_splits(B, Hkv, max_context, sm_count=None, ctas_per_sm=2, min_keys=1024):
     """Key ranges per (sequence, KV head).  The split kernel keeps ``ctas_per_sm`` CTAs resident
     per SM, so the grid B*Hkv*n runs in ceil(B*Hkv*n / (sm_count*ctas_per_sm)) waves; pick the n
-    (at least 1024 keys per range, at most 64 ranges) whose last wave is fullest, preferring
+    (at least ``min_keys`` keys per range, at most 64 ranges) whose last wave is fullest, preferring
     more ranges on a tie-ish.  Depends only on launch-time shapes (CUDA-graph safe)."""
     if sm_count is None:
         sm_count = _sm_count() if torch.cuda.is_available() else 148
     slots = sm_count * ctas_per_sm
-    n_max = int(max(1, min(64, max_context // 1024)))
+    n_max = int(max(1, min(64, max_context // min_keys)))
     best_n, best_eff = 1, -1.0
     for n in range(1, n_max + 1):
         ctas = B * Hkv * n

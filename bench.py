@@ -1093,6 +1093,10 @@ def main():
     ap.add_argument("--profile", default=None, choices=["prefill", "decode", "scan", "prep", "epilogue", "conv", "step", "prep_decode", "linear"],
                     help="run a few launches of ONE kernel on a small case (a few hundred MB, larger than L2) "
                          "and exit; meant to be wrapped in ncu")
+    ap.add_argument("--rizurax", nargs="?", const="all", default=None, metavar="KERNEL",
+                    help="instead of the default workload: throughput of the Rizurax decoder beside AtmaModel at equal size and its "
+                         "kernels beside the like ones; with a name only that kernel's leg (softmax_prefill, softmax_decode, delta_scan, "
+                         "delta_step, rows, linear)")
     args = ap.parse_args()
     if args.tokens != T_PREFILL:
         T_PREFILL = args.tokens
@@ -1105,6 +1109,15 @@ def main():
         return
     if args.profile:
         profile_case(args.profile)
+        return
+    if args.rizurax:
+        import bench_decoder
+        torch.cuda.set_device(local_rank)
+        sampler = ClockSampler(local_rank)
+        sampler.start()
+        sampler.mark_begin()
+        res = bench_decoder.run(measured_peaks(), torch.device("cuda", local_rank), None if args.rizurax == "all" else args.rizurax)
+        emit({"bench": "rizurax", "dtype": "bf16", "data": "synthetic", "peaks": measured_peaks(), **res, "clocks": sampler.stop()})
         return
     args.warmup = max(args.warmup, 3)
 
