@@ -18,8 +18,14 @@ __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
 // for results that are rounded to 16 bits anyway: the fast exponential and division (a few fp32 units in the last place)
 template <typename T>
 __device__ __forceinline__ float silu_for(float x) {
-  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
-  else return silu(x);
+  if constexpr (sizeof(T) == 2) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * x));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));        // infinity -> 0
+    return x * r;
+  } else {
+    return silu(x);
+  }
 }
 __device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
@@ -201,6 +207,130 @@ delta_prepare_kernel(const atma_delta_args a, T* __restrict__ qo, T* __restrict_
   }
 }
 
+// The same where every access is one aligned vector of CPL channels: rows travel in raw form a group of eight ahead, sums
+// are formed on channel pairs (two fp32 lanes per instruction), pointers advance by row.
+template <typename T, int CPL, int KT>
+__global__ void __launch_bounds__(128)
+delta_prepare_vec_kernel(const atma_delta_args a, T* __restrict__ qo, T* __restrict__ ko, T* __restrict__ vo, float* __restrict__ q_inv,
+                         float* __restrict__ k_inv, int run) {
+  struct alignas(CPL * sizeof(T)) Vec { T e[CPL]; };
+  constexpr int P = CPL / 2, U = 4, N = 2 * U;
+  const int lane = threadIdx.x & 31;
+  const int units = 2 * a.G + a.H;
+  const int64_t wid = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int u = (int)(wid % units);
+  const int64_t row0 = wid / units * run;
+  if (row0 >= a.total_rows) return;
+  const int row1 = (int)min((int64_t)a.total_rows, row0 + run);
+  const int nq = a.G * a.dim;
+  const int part = u < a.G ? 0 : (u < 2 * a.G ? 1 : 2);
+  const int head = part == 0 ? u : (part == 1 ? u - a.G : u - 2 * a.G);
+  const int dim = part == 2 ? a.vdim : a.dim, heads = part == 2 ? a.H : a.G;
+  const bool on = lane * CPL < dim;                             // the lanes past the head's channels work on its first ones
+  const int c0 = on ? lane * CPL : 0;
+  const int zc = part * nq + head * dim + c0;
+  const int ctot = 2 * nq + a.H * a.vdim;
+  const T* zcol = static_cast<const T*>(a.z) + zc;
+  const T* table = static_cast<const T*>(a.conv_table) + zc;
+  T* dst = (part == 0 ? qo : (part == 1 ? ko : vo)) + head * dim + c0;
+  float* inv_out = part == 0 ? q_inv : k_inv;
+  const float inv_scale = part == 0 ? a.q_scale : 1.0f;
+  const int orow = heads * dim;
+  float2 w[KT][P];
+  {
+    const T* W = static_cast<const T*>(part == 0 ? a.conv_q : (part == 1 ? a.conv_k : a.conv_v)) + ((int64_t)head * dim + c0) * KT;
+#pragma unroll
+    for (int j = 0; j < KT; ++j)
+#pragma unroll
+      for (int i = 0; i < P; ++i) w[j][i] = make_float2(to_f32(W[(2 * i) * KT + j]), to_f32(W[(2 * i + 1) * KT + j]));
+  }
+  auto unpack = [&](const Vec& x, float2 (&f)[P]) {
+#pragma unroll
+    for (int i = 0; i < P; ++i) f[i] = make_float2(to_f32(x.e[2 * i]), to_f32(x.e[2 * i + 1]));
+  };
+  for (int row = (int)row0; row < row1;) {
+    const int seq = a.row_seq[row];
+    const int first_row = a.cu_rows[seq], start = a.start_pos[seq], end = min(row1, a.cu_rows[seq + 1]);
+    const int64_t slot = a.slots[seq];
+    float2 win[KT - 1][P];
+#pragma unroll
+    for (int j = 0; j + 1 < KT; ++j) {
+      const int src = row - (KT - 1 - j), pos = start + (src - first_row);
+#pragma unroll
+      for (int i = 0; i < P; ++i) win[j][i] = make_float2(0.f, 0.f);
+      if (src >= first_row) unpack(*reinterpret_cast<const Vec*>(zcol + (int64_t)src * a.z_rs), win[j]);
+      else if (pos >= 0 && slot >= 0) unpack(*reinterpret_cast<const Vec*>(table + slot * a.conv_ss + (int64_t)(pos % KT) * ctot), win[j]);
+    }
+    const T* zp = zcol + (int64_t)row * a.z_rs;                 // the next row to request
+    T* op = dst + (int64_t)row * orow;
+    const int n = end - row;
+    Vec raw[N], nxt[N];
+#pragma unroll
+    for (int r = 0; r < N; ++r)
+      if (r < n) nxt[r] = *reinterpret_cast<const Vec*>(zp + (int64_t)r * a.z_rs);
+    for (int at = 0; at < n; at += N) {
+#pragma unroll
+      for (int r = 0; r < N; ++r) raw[r] = nxt[r];
+      zp += (int64_t)N * a.z_rs;
+#pragma unroll
+      for (int r = 0; r < N; ++r)
+        if (at + N + r < n) nxt[r] = *reinterpret_cast<const Vec*>(zp + (int64_t)r * a.z_rs);
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        float ss[U];
+#pragma unroll
+        for (int r = 0; r < U; ++r) {
+          float2 cur[P];
+          unpack(raw[g * U + r], cur);
+          Vec o;
+          ss[r] = 0.f;
+#pragma unroll
+          for (int i = 0; i < P; ++i) {
+            float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j + 1 < KT; ++j) acc = __ffma2_rn(win[j][i], w[j][i], acc);
+            acc = __ffma2_rn(cur[i], w[KT - 1][i], acc);
+            o.e[2 * i] = from_f32<T>(silu_for<T>(acc.x));
+            o.e[2 * i + 1] = from_f32<T>(silu_for<T>(acc.y));
+            const float x = to_f32(o.e[2 * i]), y = to_f32(o.e[2 * i + 1]);
+            ss[r] = fmaf(x, x, fmaf(y, y, ss[r]));
+#pragma unroll
+            for (int j = 0; j + 2 < KT; ++j) win[j][i] = win[j + 1][i];
+            win[KT - 2][i] = cur[i];
+          }
+          if (on && at + g * U + r < n) *reinterpret_cast<Vec*>(op) = o;
+          op += orow;
+          if (!on) ss[r] = 0.f;
+        }
+        if (part < 2) {
+#pragma unroll
+          for (int sft = 16; sft > 0; sft >>= 1)
+#pragma unroll
+            for (int r = 0; r < U; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], sft);
+          float mine = ss[0];
+#pragma unroll
+          for (int r = 1; r < U; ++r) mine = lane == r ? ss[r] : mine;
+          const int rr = at + g * U + lane;
+          if (lane < U && rr < n) inv_out[(int64_t)(row + rr) * a.G + head] = inv_scale / sqrtf(mine + a.unit_eps);
+        }
+      }
+    }
+    row = end;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_gates_kernel(const atma_delta_args a, float* __restrict__ log_decay, float* __restrict__ beta) {
+  const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (i >= (int64_t)a.total_rows * a.H) return;
+  const int64_t row = i / a.H;
+  const int h = (int)(i - row * a.H);
+  const T* zr = static_cast<const T*>(a.z) + row * a.z_rs + 2 * a.G * a.dim + 2 * a.H * a.vdim;
+  log_decay[i] = -expf(a.A_log[h]) * softplus(to_f32(zr[h]) + a.dt_bias[h]);
+  beta[i] = sigmoid(to_f32(zr[a.H + h]));
+}
+
 // The last `taps` inputs of every sequence into the table (its own launch: the rows above still read the old ones).
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -302,7 +432,7 @@ delta_scan_kernel(const atma_delta_args a, const T* __restrict__ q, const T* __r
 // first block's loads are in flight while the convolutions run.
 constexpr int kStepWarps = 8;
 
-template <typename T, int VEC, int RPW>
+template <typename T, int VEC, int RPW, int TAPS>             // TAPS 0: any number
 __global__ void __launch_bounds__(kStepWarps * 32)
 delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __restrict__ out, int64_t out_rs, float eps) {
   extern __shared__ float sm[];
@@ -342,22 +472,56 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
   load_state(0);
 
   // convolutions of this head's q, k and v channels
-  const int nq = a.G * K, ctot = 2 * nq + a.H * V, taps = a.taps;
+  const int nq = a.G * K, ctot = 2 * nq + a.H * V, taps = TAPS > 0 ? TAPS : a.taps;
   const T* zr = static_cast<const T*>(a.z) + b * a.z_rs;
   T* table = static_cast<T*>(a.conv_table) + slot * a.conv_ss;
   const int ring = pos % taps;
+  const int goff = 2 * nq + 2 * a.H * V;
+  const float za = to_f32(zr[goff + h]), zb = to_f32(zr[goff + a.H + h]), alog = a.A_log[h], dtb = a.dt_bias[h];
+  float gate_c = 0.f, norm_c = 0.f;              // V <= 256: one output channel per thread
+  if (tid < V) { gate_c = to_f32(zr[2 * nq + a.H * V + h * V + tid]); norm_c = to_f32(norm_w[tid]); }
+  constexpr int kRounds = 3, TA = TAPS > 0 ? TAPS : 1;           // 2 K + V <= 768 channels
   float qs = 0.f, ks = 0.f;
-  for (int i = tid; i < 2 * K + V; i += kStepWarps * 32) {
-    const int part = i < K ? 0 : (i < 2 * K ? 1 : 2);
-    const int c = i - (part == 0 ? 0 : (part == 1 ? K : 2 * K));
-    const int pc = part < 2 ? g * K + c : h * V + c;                      // channel inside the part
-    const int zc = part * nq + pc;
-    const T* w = static_cast<const T*>(part == 0 ? a.conv_q : (part == 1 ? a.conv_k : a.conv_v)) + (int64_t)pc * taps;
-    const T cur = zr[zc];
-    float acc = to_f32(cur) * to_f32(w[taps - 1]);
-    for (int j = 1; j < taps; ++j)
-      if (pos - j >= 0) acc = fmaf(to_f32(table[(int64_t)(ring - j + (ring < j ? taps : 0)) * ctot + zc]), to_f32(w[taps - 1 - j]), acc);
-    if (part == 2 || h % rep == 0) table[(int64_t)ring * ctot + zc] = cur;
+  float hist[kRounds][TA], wt[kRounds][TA];
+  auto locate = [&](int i, int& part, int& c, int& pc, int& zc) {
+    part = i < K ? 0 : (i < 2 * K ? 1 : 2);
+    c = i - part * K;
+    pc = part < 2 ? g * K + c : h * V + c;                        // channel inside the part
+    zc = part * nq + pc;
+  };
+  if constexpr (TAPS > 0) {                                        // everything requested before the first use
+#pragma unroll
+    for (int r = 0; r < kRounds; ++r) {
+      const int i = tid + r * kStepWarps * 32;
+      if (i >= 2 * K + V) continue;
+      int part, c, pc, zc;
+      locate(i, part, c, pc, zc);
+      const T* w = static_cast<const T*>(part == 0 ? a.conv_q : (part == 1 ? a.conv_k : a.conv_v)) + (int64_t)pc * TAPS;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        wt[r][j] = to_f32(w[TAPS - 1 - j]);
+        const int at = ring - j + (ring < j ? TAPS : 0);
+        hist[r][j] = j == 0 ? to_f32(zr[zc]) : (pos >= j ? to_f32(table[(int64_t)at * ctot + zc]) : 0.f);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < kRounds; ++r) {
+    const int i = tid + r * kStepWarps * 32;
+    if (i >= 2 * K + V) continue;
+    int part, c, pc, zc;
+    locate(i, part, c, pc, zc);
+    float acc = 0.f;
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(hist[r][j], wt[r][j], acc);
+    } else {
+      const T* w = static_cast<const T*>(part == 0 ? a.conv_q : (part == 1 ? a.conv_k : a.conv_v)) + (int64_t)pc * taps;
+      acc = to_f32(zr[zc]) * to_f32(w[taps - 1]);
+      for (int j = 1; j < taps; ++j)
+        if (pos >= j) acc = fmaf(to_f32(table[(int64_t)(ring - j + (ring < j ? taps : 0)) * ctot + zc]), to_f32(w[taps - 1 - j]), acc);
+    }
+    if (part == 2 || h % rep == 0) table[(int64_t)ring * ctot + zc] = zr[zc];
     const float y = round_through<T>(silu_for<T>(acc));
     if (part == 0) { s_q[c] = y; qs = fmaf(y, y, qs); }
     else if (part == 1) { s_k[c] = y; ks = fmaf(y, y, ks); }
@@ -365,9 +529,8 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
   }
   qs = warp_sum(qs); ks = warp_sum(ks);
   if (lane == 0) { s_sum[0][warp] = qs; s_sum[1][warp] = ks; }
-  const int goff = 2 * nq + 2 * a.H * V;
-  const float gm = expf(-expf(a.A_log[h]) * softplus(to_f32(zr[goff + h]) + a.dt_bias[h]));
-  const float bt = sigmoid(to_f32(zr[goff + a.H + h]));
+  const float gm = expf(-expf(alog) * softplus(za + dtb));
+  const float bt = sigmoid(zb);
   __syncthreads();
   qs = 0.f; ks = 0.f;
 #pragma unroll
@@ -427,8 +590,7 @@ delta_step_kernel(const atma_delta_args a, const T* __restrict__ norm_w, T* __re
 #pragma unroll
   for (int i = 0; i < kStepWarps; ++i) osq += s_sum[2][i];
   const float rs = 1.0f / sqrtf(osq / (float)V + eps);
-  const T* gate = zr + 2 * nq + a.H * V + h * V;
-  for (int c = tid; c < V; c += kStepWarps * 32) orow[c] = from_f32<T>(s_o[c] * rs * to_f32(norm_w[c]) * silu(to_f32(gate[c])));
+  if (tid < V) orow[tid] = from_f32<T>(s_o[tid] * rs * norm_c * silu_for<T>(gate_c));
 }
 
 int check(const atma_delta_args* a, const char* what) {
@@ -447,6 +609,20 @@ int launch_prepare(const atma_delta_args& a, void* q, void* k, void* v, float* q
   const int run = a.total_rows >= kLongRows ? kRunLong : kRunShort;
   const int64_t warps = (int64_t)((a.total_rows + run - 1) / run) * (2 * a.G + a.H + 1);
   const unsigned grid = (unsigned)((warps + 3) / 4);
+  auto al = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
+  if constexpr (CPL > 1) {
+    if (a.taps >= 2 && a.taps <= 4 && a.dim % CPL == 0 && a.vdim % CPL == 0 && a.z_rs % CPL == 0 && a.conv_ss % CPL == 0 && al(a.z) &&
+        al(a.conv_table) && al(q) && al(k) && al(v)) {
+      const unsigned vgrid = (unsigned)(((int64_t)((a.total_rows + run - 1) / run) * (2 * a.G + a.H) + 3) / 4);
+#define ATMA_PREPV(KT) delta_prepare_vec_kernel<T, CPL, KT><<<vgrid, 128, 0, st>>>(a, (T*)q, (T*)k, (T*)v, qi, ki, run)
+      if (a.taps == 2) ATMA_PREPV(2); else if (a.taps == 3) ATMA_PREPV(3); else ATMA_PREPV(4);
+#undef ATMA_PREPV
+      delta_gates_kernel<T><<<(unsigned)(((int64_t)a.total_rows * a.H + 255) / 256), 256, 0, st>>>(a, ld, bt);
+      const int ct = 2 * a.G * a.dim + a.H * a.vdim;
+      delta_conv_state_kernel<T><<<dim3((ct + 255) / 256, a.n_seqs), 256, 0, st>>>(a, ct);
+      return launch_status("delta_prepare");
+    }
+  }
 #define ATMA_PREP(KT) delta_prepare_kernel<T, CPL, KT><<<grid, 128, 0, st>>>(a, (T*)q, (T*)k, (T*)v, qi, ki, ld, bt, run)
   switch (a.taps) {
     case 2: ATMA_PREP(2); break;
@@ -487,9 +663,11 @@ int step_t(const atma_delta_args& a, const void* w, void* out, int64_t out_rs, f
   const dim3 grid(a.H, a.n_seqs);
   const int smem = (2 * a.dim + 2 * a.vdim) * 4;
   const bool vec = a.vdim % 4 == 0 && a.state_ss % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state_table) & 15) == 0;
-#define ATMA_STEP(V, R) delta_step_kernel<T, V, R><<<grid, kStepWarps * 32, smem, st>>>(a, (const T*)w, (T*)out, out_rs, eps)
+#define ATMA_STEPT(V, R, K) delta_step_kernel<T, V, R, K><<<grid, kStepWarps * 32, smem, st>>>(a, (const T*)w, (T*)out, out_rs, eps)
+#define ATMA_STEP(V, R) do { if (a.taps == 4) ATMA_STEPT(V, R, 4); else ATMA_STEPT(V, R, 0); } while (0)
   if (vec) { if (a.dim <= 64) ATMA_STEP(4, 8); else if (a.dim <= 128) ATMA_STEP(4, 16); else ATMA_STEP(4, 32); }
   else { if (a.dim <= 64) ATMA_STEP(1, 8); else if (a.dim <= 128) ATMA_STEP(1, 16); else ATMA_STEP(1, 32); }
+#undef ATMA_STEPT
 #undef ATMA_STEP
   return launch_status("delta_step");
 }

@@ -19,7 +19,8 @@
 //   terms, the B operands are the K and Q rows exactly as TMA delivers them and M1, M2 as two terms.  Issue order per
 //   chunk: P = S^T K^T | first half of S^T Q^T | U^T = R^T M1^T | second half of S^T Q^T | dS^T = U^T K | R^T M2^T, so that
 //   the products the next step does not wait for run under the thread phases.
-//     warp 0 TMA producer (two stages), warp 1 MMA issuer, warps 2-9 state warps (lane quarter warp % 4, column half).
+//     warp 0 TMA producer (two stages), warp 1 MMA issuer, warps 2-17 state warps (TMEM lanes 32 (warp % 4) .. + 31, column
+//     quarter (warp - 2) / 4); what a thread phase reads from shared memory is fetched while the product before it runs.
 //     TMEM: S hi/lo [0,128) | P, U [128,192) | dS [192,320) | R hi/lo [320,384) | U hi/lo, then R M2 [384,448) | S Q [448,512)
 // Every mbarrier wait is bounded; on expiry a CTA frees its TMEM, returns and leaves a status word for the host.
 #include "delta_rule.cuh"
@@ -399,7 +400,7 @@ delta_factors_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
 }
 
 // ======================================= recurrence =======================================================================
-constexpr int kStages = 2;
+constexpr int kStages = 2, kStateWarps = 16, kRecurThreads = 64 + 32 * kStateWarps;
 // a stage: [K rows; Q rows] as two boxes of 64 channels x 128 rows | V, two boxes of 64 channels x 64 rows | [M1; M2] rounded,
 // [M1; M2] remainders | scalars
 constexpr int kOffKQ = 0, kOffRV = 32768, kOffRM = 49152, kOffRS = 81920, kStageBytes = 82944;
@@ -411,7 +412,7 @@ struct RecurBarriers {
   uint64_t s_ready, pq_full, r_ready, uo_full, us_ready, s_done;
 };
 
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kRecurThreads, 1)
 delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                    const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_m, const Params p) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -430,8 +431,8 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int64_t rec0 = (int64_t)h * p.NC + c0;
 
   if (tid == 0) {
-    for (int i = 0; i < kStages; ++i) { mbar_init(&bar.in_full[i], 1); mbar_init(&bar.m_full[i], 1); mbar_init(&bar.empty[i], 9); }
-    mbar_init(&bar.s_ready, 8); mbar_init(&bar.r_ready, 8); mbar_init(&bar.us_ready, 8);
+    for (int i = 0; i < kStages; ++i) { mbar_init(&bar.in_full[i], 1); mbar_init(&bar.m_full[i], 1); mbar_init(&bar.empty[i], 1 + kStateWarps); }
+    mbar_init(&bar.s_ready, kStateWarps); mbar_init(&bar.r_ready, kStateWarps); mbar_init(&bar.us_ready, kStateWarps);
     mbar_init(&bar.pq_full, 1); mbar_init(&bar.uo_full, 1); mbar_init(&bar.s_done, 1);
     s_abort = 0;
     fence_barrier_init();
@@ -517,19 +518,19 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     __syncwarp();
   } else {
     // ---- state warps -------------------------------------------------------------------------------------------
-    const int quad = warp & 3, half = (warp - 2) >> 2;
+    const int quad = warp & 3, qt = (warp - 2) >> 2;   // qt: 32 of the 128 state columns, 16 of a chunk's 64 rows
     const int v = 32 * quad + lane;                    // TMEM lane = value channel of this CTA's block
     const uint32_t lane_base = tbase + (uint32_t(32 * quad) << 16);
     const int vcol = (hv % vblocks) * kD + v;
-    float* plane = p.state + slot * p.state_ss + ((int64_t)h * kD + 64 * half) * p.vdim + vcol;   // element (k = 64 half + j, v)
+    float* plane = p.state + slot * p.state_ss + ((int64_t)h * kD + 32 * qt) * p.vdim + vcol;   // element (k = 32 qt + j, v)
     const bool fresh = p.start_pos[b] == 0;
-    float S[64];
+    float S[32];
     {
       const float* src = plane;
       int64_t step = p.vdim;
-      asm volatile("" : "+l"(step));
+      asm volatile("" : "+l"(step));                    // not a loop invariant: its multiples would be kept in registers
 #pragma unroll
-      for (int j = 0; j < 64; ++j) { S[j] = fresh ? 0.f : *src; src += step; }
+      for (int j = 0; j < 32; ++j) { S[j] = fresh ? 0.f : *src; src += step; }
     }
     float gC = 0.f;                                    // decay over the chunk before
     bool ok = true;
@@ -539,23 +540,19 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
+        uint32_t d[32];
+        tmem_ld32(lane_base + kColD + 32 * qt, d);
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          uint32_t d[32];
-          tmem_ld32(lane_base + kColD + 64 * half + 32 * q, d);
-#pragma unroll
-          for (int j = 0; j < 32; ++j) S[32 * q + j] = fmaf(gC, S[32 * q + j], __uint_as_float(d[j]));
-        }
+        for (int j = 0; j < 32; ++j) S[j] = fmaf(gC, S[j], __uint_as_float(d[j]));
       }
       if (i == n_chunks) break;
       // ---- S^T as two 16-bit terms (the dS columns have been read: the next products may overwrite them) ----
-#pragma unroll
-      for (int q = 0; q < 2; ++q) {
+      {
         uint32_t hi[16], lo[16];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) split2(S[32 * q + 2 * j], S[32 * q + 2 * j + 1], hi[j], lo[j]);
-        tmem_st16(lane_base + kColS + 32 * half + 16 * q, hi);
-        tmem_st16(lane_base + kColS + 64 + 32 * half + 16 * q, lo);
+        for (int j = 0; j < 16; ++j) split2(S[2 * j], S[2 * j + 1], hi[j], lo[j]);
+        tmem_st16(lane_base + kColS + 16 * qt, hi);
+        tmem_st16(lane_base + kColS + 64 + 16 * qt, lo);
       }
       tmem_st_wait();
       tc_fence_before();
@@ -564,61 +561,63 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 
       const int s = i % kStages;
       const uint8_t* st = smem + s * kStageBytes;
-      const float* sc = reinterpret_cast<const float*>(st + kOffRS);
-      // ---- R^T = V^T - (a k_inv) P: this thread's value channel, rows 32 half .. + 31 ----
-      ok = mbar_wait(&bar.in_full[s], (uint32_t)(i / kStages) & 1u, abort_flag) && mbar_wait(&bar.pq_full, (uint32_t)i & 1u, abort_flag);
+      const float* sc = reinterpret_cast<const float*>(st + kOffRS) + 16 * qt;
+      // ---- R^T = V^T - (a k_inv) P: this thread's value channel, rows 16 qt .. + 15 ----
+      ok = mbar_wait(&bar.in_full[s], (uint32_t)(i / kStages) & 1u, abort_flag);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      float vv[16], ek[16];
+      {
+        const uint8_t* vb = st + kOffRV + (v >> 6) * 8192 + (v & 7) * 2;
+        const int ch = (v & 63) >> 3;
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          const int t = 16 * qt + j;
+          vv[j] = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vb + t * 128 + ((ch ^ (t & 7)) << 4)));
+        }
+#pragma unroll
+        for (int j = 0; j < 16; j += 4) {
+          const float4 e = *reinterpret_cast<const float4*>(sc + j);
+          ek[j] = e.x; ek[j + 1] = e.y; ek[j + 2] = e.z; ek[j + 3] = e.w;
+        }
+      }
+      ok = mbar_wait(&bar.pq_full, (uint32_t)i & 1u, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
       {
-        const uint8_t* vb = st + kOffRV + (v >> 6) * 8192 + (v & 7) * 2;
-        const int ch = (v & 63) >> 3;
-        uint32_t pr[32], hi[16], lo[16];
-        tmem_ld32(lane_base + kColP + 32 * half, pr);
+        uint32_t pr[16], hi[8], lo[8];
+        tmem_ld16(lane_base + kColP + 16 * qt, pr);
 #pragma unroll
-        for (int j = 0; j < 32; j += 4) {
-          const float4 ek = *reinterpret_cast<const float4*>(sc + 32 * half + j);
-          const float e[4] = {ek.x, ek.y, ek.z, ek.w};
-          float x[4];
-#pragma unroll
-          for (int q = 0; q < 4; ++q) {
-            const int t = 32 * half + j + q;
-            const float vv = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vb + t * 128 + ((ch ^ (t & 7)) << 4)));
-            x[q] = fmaf(-e[q], __uint_as_float(pr[j + q]), vv);
-          }
-          split2(x[0], x[1], hi[j >> 1], lo[j >> 1]);
-          split2(x[2], x[3], hi[(j >> 1) + 1], lo[(j >> 1) + 1]);
-        }
-        tmem_st16(lane_base + kColR + 16 * half, hi);
-        tmem_st16(lane_base + kColR + 32 + 16 * half, lo);
+        for (int j = 0; j < 16; j += 2)
+          split2(fmaf(-ek[j], __uint_as_float(pr[j]), vv[j]), fmaf(-ek[j + 1], __uint_as_float(pr[j + 1]), vv[j + 1]), hi[j >> 1], lo[j >> 1]);
+        tmem_st8(lane_base + kColR + 8 * qt, hi);
+        tmem_st8(lane_base + kColR + 32 + 8 * qt, lo);
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&bar.r_ready);
       }
       // ---- U^T scaled by (a_C / a) k_inv; S^T Q^T leaves the columns that dS will take ----
+      float ed[16];
+#pragma unroll
+      for (int j = 0; j < 16; j += 4) {
+        const float4 e = *reinterpret_cast<const float4*>(sc + 128 + j);
+        ed[j] = e.x; ed[j + 1] = e.y; ed[j + 2] = e.z; ed[j + 3] = e.w;
+      }
+      uint32_t sq[16];
+      tmem_ld16(lane_base + kColQ + 16 * qt, sq);
       ok = mbar_wait(&bar.uo_full, (uint32_t)i & 1u, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      uint32_t sq[32];
-      tmem_ld32(lane_base + kColQ + 32 * half, sq);
       {
-        uint32_t hi[16], lo[16];
+        uint32_t u[16], hi[8], lo[8];
+        tmem_ld16(lane_base + kColX + 16 * qt, u);
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          uint32_t u[16];
-          tmem_ld16(lane_base + kColX + 32 * half + 16 * q, u);
-#pragma unroll
-          for (int j = 0; j < 16; j += 4) {
-            const float4 ed = *reinterpret_cast<const float4*>(sc + 128 + 32 * half + 16 * q + j);
-            const int w = (16 * q + j) >> 1;
-            split2(__uint_as_float(u[j]) * ed.x, __uint_as_float(u[j + 1]) * ed.y, hi[w], lo[w]);
-            split2(__uint_as_float(u[j + 2]) * ed.z, __uint_as_float(u[j + 3]) * ed.w, hi[w + 1], lo[w + 1]);
-          }
-        }
-        tmem_st16(lane_base + kColU + 16 * half, hi);
-        tmem_st16(lane_base + kColU + 32 + 16 * half, lo);
+        for (int j = 0; j < 16; j += 2) split2(__uint_as_float(u[j]) * ed[j], __uint_as_float(u[j + 1]) * ed[j + 1], hi[j >> 1], lo[j >> 1]);
+        tmem_st8(lane_base + kColU + 8 * qt, hi);
+        tmem_st8(lane_base + kColU + 32 + 8 * qt, lo);
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -626,32 +625,22 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       }
       // ---- O = (a q_inv) S Q + R M2, under the last product ----
       {
-        gC = sc[192];
-        const int t0 = row_begin + i * kC + 32 * half;
-        const int n_ok = min(32, row_end - t0);
+        gC = reinterpret_cast<const float*>(st + kOffRS)[192];
+        const int t0 = row_begin + i * kC + 16 * qt;
+        const int n_ok = min(16, row_end - t0);
         uint16_t* oc = static_cast<uint16_t*>(p.o) + ((int64_t)t0 * p.H + h) * p.vdim + vcol;
         int64_t orow = (int64_t)p.H * p.vdim;
-        asm volatile("" : "+l"(orow));                  // not a loop invariant: its 31 multiples would be kept in registers
+        asm volatile("" : "+l"(orow));
+        uint32_t r[16];
+        tmem_ld16(lane_base + kColX2 + 16 * qt, r);
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          uint32_t r[16];
-          tmem_ld16(lane_base + kColX2 + 32 * half + 16 * q, r);
-#pragma unroll
-          for (int j = 0; j < 16; j += 4) {
-            const float4 e = *reinterpret_cast<const float4*>(sc + 64 + 32 * half + 16 * q + j);
-            const uint32_t w0 = pack_bf16(fmaf(e.x, __uint_as_float(sq[16 * q + j]), __uint_as_float(r[j])),
-                                          fmaf(e.y, __uint_as_float(sq[16 * q + j + 1]), __uint_as_float(r[j + 1])));
-            const uint32_t w1 = pack_bf16(fmaf(e.z, __uint_as_float(sq[16 * q + j + 2]), __uint_as_float(r[j + 2])),
-                                          fmaf(e.w, __uint_as_float(sq[16 * q + j + 3]), __uint_as_float(r[j + 3])));
-            if (16 * q + j < n_ok) *oc = (uint16_t)(w0 & 0xffffu);
-            oc += orow;
-            if (16 * q + j + 1 < n_ok) *oc = (uint16_t)(w0 >> 16);
-            oc += orow;
-            if (16 * q + j + 2 < n_ok) *oc = (uint16_t)(w1 & 0xffffu);
-            oc += orow;
-            if (16 * q + j + 3 < n_ok) *oc = (uint16_t)(w1 >> 16);
-            oc += orow;
-          }
+        for (int j = 0; j < 16; j += 2) {
+          const float2 e = *reinterpret_cast<const float2*>(sc + 64 + j);
+          const uint32_t w = pack_bf16(fmaf(e.x, __uint_as_float(sq[j]), __uint_as_float(r[j])), fmaf(e.y, __uint_as_float(sq[j + 1]), __uint_as_float(r[j + 1])));
+          if (j < n_ok) *oc = (uint16_t)(w & 0xffffu);
+          oc += orow;
+          if (j + 1 < n_ok) *oc = (uint16_t)(w >> 16);
+          oc += orow;
         }
         tc_fence_before();
         __syncwarp();
@@ -660,9 +649,9 @@ delta_recur_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     }
     if (ok) {
       int64_t step = p.vdim;
-      asm volatile("" : "+l"(step));                    // opaque, like orow
+      asm volatile("" : "+l"(step));
 #pragma unroll
-      for (int j = 0; j < 64; ++j) { *plane = S[j]; plane += step; }
+      for (int j = 0; j < 32; ++j) { *plane = S[j]; plane += step; }
     }
   }
   tc_fence_before();
@@ -727,7 +716,7 @@ int delta_scan_sm100(const atma_delta_args& a, const void* q, const void* k, con
   ATMA_CUDA_OK(cudaFuncSetAttribute(delta_factors_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFactorSmem));
   delta_factors_kernel<<<(unsigned)(tiles < 2 * sms ? tiles : 2 * sms), kThreads, kFactorSmem, st>>>(mq, mk, p);
   ATMA_CUDA_OK(cudaFuncSetAttribute(delta_recur_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kRecurSmem));
-  delta_recur_kernel<<<dim3(a.H * (a.vdim / kD), a.n_seqs), kThreads, kRecurSmem, st>>>(mq, mk, mv, mm, p);
+  delta_recur_kernel<<<dim3(a.H * (a.vdim / kD), a.n_seqs), kRecurThreads, kRecurSmem, st>>>(mq, mk, mv, mm, p);
   return launch_status("delta_scan (tcgen05)");
 }
 

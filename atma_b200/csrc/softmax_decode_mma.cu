@@ -128,13 +128,17 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     if (it + STAGES - 1 < n_tiles) load_tile(it + STAGES - 1);
     cp_async_commit();
     const uint32_t Ksm = smem_u32(sm + (it % STAGES) * kStage), Vsm = Ksm + kKBytes;
-    float S[4] = {0.f, 0.f, 0.f, 0.f};
+    float S[4] = {0.f, 0.f, 0.f, 0.f}, S2[4] = {0.f, 0.f, 0.f, 0.f};      // two chains, half as long
 #pragma unroll
-    for (int ks = 0; ks < KS; ++ks) {
-      uint32_t af[4];
+    for (int ks = 0; ks < KS; ks += 2) {
+      uint32_t af[4], ag[4];
       ldsm_x4(Ksm + tile_off(16 * warp + am, 16 * ks + ak, KD), af);
+      ldsm_x4(Ksm + tile_off(16 * warp + am, 16 * ks + 16 + ak, KD), ag);
       mma16816<true>(S, af, qb[ks][0], qb[ks][1]);
+      mma16816<true>(S2, ag, qb[ks + 1][0], qb[ks + 1][1]);
     }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) S[e] += S2[e];
     const int key0 = lo + it * kTileKeys + 16 * warp + gq;
     const bool ok0 = key0 < hi, ok1 = key0 + 8 < hi;
     float x[4];                               // [key gq][e], [key gq + 8][e]
@@ -165,11 +169,14 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     const uint32_t pb0 = movmatrix_trans(h01), pb1 = movmatrix_trans(h23);
     const uint32_t lb0 = movmatrix_trans(pack2<true>(p[0] - f01.x, p[1] - f01.y)), lb1 = movmatrix_trans(pack2<true>(p[2] - f23.x, p[3] - f23.y));
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      uint32_t af[4];
-      ldsm_x4_trans(Vsm + tile_off(16 * warp + vk, 16 * mt + vm, VD), af);
-      mma16816<true>(O[mt], af, pb0, pb1);
-      mma16816<true>(O[mt], af, lb0, lb1);
+    for (int mt = 0; mt < MT; mt += 4) {
+      uint32_t af[4][4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) ldsm_x4_trans(Vsm + tile_off(16 * warp + vk, 16 * (mt + q) + vm, VD), af[q]);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) mma16816<true>(O[mt + q], af[q], pb0, pb1);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) mma16816<true>(O[mt + q], af[q], lb0, lb1);
     }
   }
   cp_async_wait<0>();
