@@ -276,3 +276,18 @@ def test_command_line_arguments():
     from atma_b200.generate import ids, parse_args
     a = parse_args(["--model", "m", "--prompt", "1,2", "--prompt", "3", "--top-k", "4"])
     assert [ids(p) for p in a.prompt] == [[1, 2], [3]] and a.top_k == 4 and a.temperature == 0.0
+
+
+def test_prefill_attention_register_hand_over_fits_the_launch_pool():
+    """What setmaxnreg asks for must add up to no more than the CTA is launched with, or the last request never returns."""
+    import os
+    import re
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    log = os.path.join(root, "atma_b200", "build", "softmax_prefill_sm100.o.log")
+    src = open(os.path.join(root, "atma_b200", "csrc", "softmax_prefill_sm100.cu")).read()
+    if not os.path.exists(log):
+        pytest.skip("no compiler report (the library was not built in this tree)")
+    used = [int(x) for x in re.findall(r"Used (\d+) registers", open(log).read())]
+    threads = int(re.search(r"kThreads = (\d+)", src).group(1))
+    dec, inc = (int(re.search(rf"setmaxnreg\.{w}\.sync\.aligned\.u32 (\d+);", src).group(1)) for w in ("dec", "inc"))
+    assert used and threads % 128 == 0 and all(dec * 128 + inc * (threads - 128) <= n * threads for n in used)
