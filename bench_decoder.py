@@ -43,7 +43,7 @@ def rizurax_config(width, layers):
     delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}
     att = {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.4, "scale": 0.125, "rot": rot}}
     return {"architecture": "Rizurax", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "layers": [att if i % 4 == 2 else delta for i in range(layers)],
-            "embedding": {"bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 17}}}
+            "embedding": {"bigram": {"buckets": 4093, "mul_prev": 101, "mul_cur": 7}}}
 
 
 def rizurax_weights(cfg, seed, device):
@@ -277,7 +277,7 @@ def kernel_legs(peaks, device, only=None):
         out["gelu_gate"] = {"shape": f"{n // 2} x {2 * D}", "rizurax": roof(ms, peaks, 3.0 * o.numel() * 2), "like": ["squared_relu_gate", roof(lk, peaks, 3.0 * o.numel() * 2)]}
         ids, prev = torch.randint(0, VOCAB, (n,), device=device, dtype=torch.int32), torch.randint(0, VOCAB, (n,), device=device, dtype=torch.int32)
         e, bg = rnd(VOCAB, D), rnd(4094, D)
-        ms = dev_ms(lambda: ops.embed_bigram(ids, prev, e, bg, 31, 17))
+        ms = dev_ms(lambda: ops.embed_bigram(ids, prev, e, bg, 101, 7))
         lk = dev_ms(lambda: e[ids.long()])
         out["embed_bigram"] = {"shape": f"{n} x {D}", "rizurax": roof(ms, peaks, n * D * 8.0), "like": ["embedding gather (torch)", roof(lk, peaks, n * D * 4.0)]}
         del x, y, gu

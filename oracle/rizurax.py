@@ -1,7 +1,7 @@
 """Plain CPU restatement of the Rizurax decoder, one function per mechanism.  TEST INFRASTRUCTURE ONLY.
 
-Whole sequences from their first token, no cache, no chunks, no shared code with the product path: the checker for
-the kernels and for the engine.  Every function takes and returns ordinary torch tensors (fp32 or fp64); loops run
+Whole sequences from their first token, no cache, no chunks, no shared code with the product path: what
+the tests compare the kernels and the engine with.  Every function takes and returns ordinary torch tensors (fp32 or fp64); loops run
 over tokens and heads exactly as the equations are written.  ``w`` is a mapping from tensor names to tensors, ``cfg``
 the parsed config.json.
 """
