@@ -71,6 +71,7 @@ class SoftmaxArgs(Structure):
         ("H", c_int), ("G", c_int), ("maps", c_int), ("dim", c_int), ("vdim", c_int),
         ("num_blocks", c_int), ("block_size", c_int), ("max_blocks", c_int), ("n_splits", c_int), ("dtype", c_int),
         ("scale", c_float), ("lambda_", c_float), ("out_scale", c_float), ("eps", c_float),
+        ("gate", c_void_p), ("gate_rs", c_int64), ("window", c_int), ("keep_first", c_int), ("sink", c_float),
     ]
 
 
@@ -165,6 +166,11 @@ _DECODER_SIGNATURES = {
     "atma_decoder_device_status": (c_int, [POINTER(c_int)]),
     "atma_embed_bigram": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int, c_void_p]),
     "atma_residual_norms": (c_int, [c_void_p] * 7 + [c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "atma_embed_position_norm": (c_int, [c_void_p] * 7 + [c_int] * 4 + [c_float] * 3 + [c_int, c_void_p]),
+    "atma_residual_post_norm": (c_int, [c_void_p] * 7 + [c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "atma_bias_squared_relu": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
+    "atma_norm_store": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_float, c_float] + [c_void_p] * 3 +
+                        [c_int] * 5 + [c_void_p]),
     "atma_gelu_gate": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
     "atma_head_norm_silu_gate": (c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_float,
                                          c_int, c_void_p]),

@@ -23,7 +23,7 @@ LIBS = {"b200": os.path.join(HERE, "libatma_b200.so"), "decoder": os.path.join(H
 LIB = LIBS["b200"]
 
 SHARED = {"error.cu", "sm100_host.cu", "decode_linear.cu"}
-DECODER = {"decoder_rows.cu", "rotary_store.cu", "softmax_attention.cu", "softmax_prefill_sm100.cu", "softmax_decode_mma.cu",
+DECODER = {"decoder_rows.cu", "norm_store.cu", "rotary_store.cu", "softmax_attention.cu", "softmax_prefill_sm100.cu", "softmax_decode_mma.cu",
            "delta_rule.cu", "delta_scan_sm100.cu"}
 
 NVCC_FLAGS = [

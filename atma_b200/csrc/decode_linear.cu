@@ -23,18 +23,19 @@ struct LinArgs {
   const void* x; int64_t x_rs;             // [B][K]
   const void* w;                           // [N][K] row-major (torch Linear layout)
   const void* bias;                        // [N] or null
-  void* out; int64_t out_rs;               // [B][N] (plain) or [B][N/2] (gated)
+  void* out; int64_t out_rs;               // [B][N], or [B][N/2] where two halves are combined
   int B, N, K;
   int ks;                                  // K splits per unit (power of two <= 16); units per CTA = 16 / ks
-  int units;                               // 16-feature units (gated: N/2/16, else N/16)
+  int units;                               // 16-feature units (two halves: N/2/16, else N/16)
 };
 
 // One warp: its unit's rows [row0, row0+16) (and, gated, [row0 + N/2, ...)) over k in [k0, k1).
-template <typename T, int NT, int kGated>                  // kGated: 0 plain, 1 up * relu(gate)^2, 2 gelu_tanh(gate) * up
+// kGated: 0 plain, 1 up * relu(gate)^2, 2 gelu_tanh(gate) * up, 3 relu(y)^2 of every feature (no second half)
+template <typename T, int NT, int kGated>
 __global__ void __launch_bounds__(kWarps * 32)
 decode_linear_kernel(const LinArgs a) {
   constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
-  constexpr int kTiles = kGated != 0 ? 2 : 1;
+  constexpr int kTiles = kGated == 1 || kGated == 2 ? 2 : 1;
   __shared__ float part[kWarps][kTiles][NT][4][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -136,6 +137,9 @@ decode_linear_kernel(const LinArgs a) {
         float sq = p * p;
         if constexpr (kBf16) sq = round_through<T>(sq);         // eager bf16 materialises relu(x)^2 before the multiply
         v = y[1][j] * sq;
+      } else if constexpr (kGated == 3) {
+        const float p = fmaxf(y[0][j], 0.f);
+        v = p * p;
       }
       out[(int64_t)b * a.out_rs + feat] = from_f32<T>(v);
     }
@@ -152,14 +156,16 @@ extern "C" int atma_decode_linear(const void* x, int64_t x_row_stride, const voi
   ATMA_REQUIRE(dtype == ATMA_BF16 || dtype == ATMA_F16, "decode_linear: 16-bit activations and weights only (dtype %d)", dtype);
   ATMA_REQUIRE(B >= 0 && B <= kMaxRows, "decode_linear: %d rows; this entry serves decode batches of up to %d", B, kMaxRows);
   ATMA_REQUIRE(K >= 32 && K % 32 == 0, "decode_linear: K=%d must be a multiple of 32", K);
-  ATMA_REQUIRE(N > 0 && N % (gated ? 32 : 16) == 0, "decode_linear: N=%d must be a multiple of %d", N, gated ? 32 : 16);
+  ATMA_REQUIRE(gated >= 0 && gated <= 3, "decode_linear: unknown form %d", gated);
+  const bool halves = gated == 1 || gated == 2;
+  ATMA_REQUIRE(N > 0 && N % (halves ? 32 : 16) == 0, "decode_linear: N=%d must be a multiple of %d", N, halves ? 32 : 16);
   ATMA_REQUIRE((reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(weight) & 15) == 0 && x_row_stride % 8 == 0,
                "decode_linear: x and weight must be 16-byte aligned with a row stride that is a multiple of 8 elements");
   if (B == 0) return ATMA_OK;
   LinArgs a{};
   a.x = x; a.x_rs = x_row_stride; a.w = weight; a.bias = bias; a.out = out; a.out_rs = out_row_stride;
   a.B = B; a.N = N; a.K = K;
-  a.units = (gated ? N / 2 : N) / 16;
+  a.units = (halves ? N / 2 : N) / 16;
   // K splits per unit: as many as give every split whole 32-k blocks and keep the grid within one wave
   const int sms = sm_count_of_current_device();
   int ks = kWarps;
@@ -171,7 +177,8 @@ extern "C" int atma_decode_linear(const void* x, int64_t x_row_stride, const voi
 #define ATMA_LIN(T, NT, G) decode_linear_kernel<T, NT, G><<<grid, block, 0, st>>>(a)
 #define ATMA_LIN_ANY(T, NT)                                                                  \
   do {                                                                                       \
-    if (gated == 2) ATMA_LIN(T, NT, 2); else if (gated) ATMA_LIN(T, NT, 1); else ATMA_LIN(T, NT, 0); \
+    if (gated == 3) ATMA_LIN(T, NT, 3); else if (gated == 2) ATMA_LIN(T, NT, 2);            \
+    else if (gated) ATMA_LIN(T, NT, 1); else ATMA_LIN(T, NT, 0);                             \
   } while (0)
   if (dtype == ATMA_BF16) {
     if (B <= 8) ATMA_LIN_ANY(__nv_bfloat16, 1); else ATMA_LIN_ANY(__nv_bfloat16, 2);

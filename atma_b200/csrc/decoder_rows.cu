@@ -1,6 +1,6 @@
-// Row operations of the decoder models: token + bigram embedding, the fp32 residual stream with its zero-centred
-// RMS norms, the gelu-gated feed-forward product and the per-head norm with a silu gate.  Everything is one pass
-// over rows, 16 bytes per thread and access where the shapes allow it.
+// Row operations of the decoder models: token + bigram and token + learned-position embeddings, the fp32 residual
+// stream with RMS norms of the stream or of what a sublayer adds to it, the feed-forward activations and the per-head
+// norm with a silu gate.  Everything is one pass over rows, 16 bytes per thread and access where the shapes allow it.
 #include "common.cuh"
 #include "../../include/atma_decoder.h"
 
@@ -118,6 +118,191 @@ residual_norms_any_kernel(const float* x, const T* __restrict__ y, float* x_out,
   }
 }
 
+// ---- rows that are normalised before they enter the residual stream -----------------------------------
+// Sum over the CTA, the same value in every thread.  Two calls use different halves of s_part.
+__device__ __forceinline__ float cta_sum(float v, float* s_part) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) s_part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) tot += s_part[i];
+  return tot;
+}
+
+// Loads and stores of VEC (4 or 1) consecutive channels as fp32.
+template <int VEC>
+__device__ __forceinline__ void load_f32(const float* p, float (&f)[VEC]) {
+  const Pack<float, VEC> v = *reinterpret_cast<const Pack<float, VEC>*>(p);
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) f[e] = v.e[e];
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void load_t(const T* p, float (&f)[VEC]) {
+  const Pack<T, VEC> v = *reinterpret_cast<const Pack<T, VEC>*>(p);
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) f[e] = to_f32(v.e[e]);
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_t(T* p, const float (&f)[VEC]) {
+  Pack<T, VEC> v;
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) v.e[e] = from_f32<T>(f[e]);
+  *reinterpret_cast<Pack<T, VEC>*>(p) = v;
+}
+
+struct EmbedNormArgs {
+  const int32_t *ids, *positions;
+  const void *embed, *pos, *w;
+  float* x;
+  void* h;
+  int D, vocab, max_positions;
+  float scale, eps, offset;
+};
+
+// One CTA per row, up to NV groups of VEC channels per thread held between the sum of squares and the result.
+template <typename T, int VEC, int NV>
+__global__ void __launch_bounds__(kNormThreads)
+embed_position_norm_kernel(const EmbedNormArgs a) {
+  __shared__ float s_part[kNormThreads / 32];
+  const int64_t row = blockIdx.x;
+  const T* e = static_cast<const T*>(a.embed) + (int64_t)min(max(a.ids[row], 0), a.vocab - 1) * a.D;
+  const T* p = a.pos == nullptr ? nullptr : static_cast<const T*>(a.pos) + (int64_t)min(max(a.positions[row], 0), a.max_positions - 1) * a.D;
+  const T* w = static_cast<const T*>(a.w);
+  float v[NV][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= a.D) continue;
+    load_t<T, VEC>(e + c, v[i]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[i][k] *= a.scale;
+    if (p != nullptr) {
+      float q[VEC];
+      load_t<T, VEC>(p + c, q);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[i][k] += q[k];
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+  }
+  const float rs = 1.0f / sqrtf(cta_sum(ss, s_part) / (float)a.D + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= a.D) continue;
+    float g[VEC];
+    load_t<T, VEC>(w + c, g);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[i][k] = v[i][k] * rs * (a.offset + g[k]);
+    store_t<float, VEC>(a.x + row * a.D + c, v[i]);
+    if (a.h != nullptr) store_t<T, VEC>(static_cast<T*>(a.h) + row * a.D + c, v[i]);
+  }
+}
+
+struct PostNormArgs {
+  const float* x;
+  const void *y, *bias, *w;
+  float* x_out;
+  void* h;
+  const void* w_next;
+  int D;
+  float eps, offset;
+};
+
+template <typename T, int VEC, int NV>
+__global__ void __launch_bounds__(kNormThreads)
+residual_post_norm_kernel(const PostNormArgs a) {
+  __shared__ float s_part[2][kNormThreads / 32];
+  const int64_t base = (int64_t)blockIdx.x * a.D;
+  const T *y = static_cast<const T*>(a.y) + base, *bias = static_cast<const T*>(a.bias), *w = static_cast<const T*>(a.w);
+  float v[NV][VEC], x[NV][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= a.D) continue;
+    load_t<T, VEC>(y + c, v[i]);
+    load_f32<VEC>(a.x + base + c, x[i]);
+    if (bias != nullptr) {
+      float b[VEC];
+      load_t<T, VEC>(bias + c, b);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[i][k] += b[k];
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+  }
+  const float rs = 1.0f / sqrtf(cta_sum(ss, s_part[0]) / (float)a.D + a.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= a.D) continue;
+    float g[VEC];
+    load_t<T, VEC>(w + c, g);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+      x[i][k] = fmaf(v[i][k] * rs, a.offset + g[k], x[i][k]);
+      ss = fmaf(x[i][k], x[i][k], ss);
+    }
+    if (a.x_out != nullptr) store_t<float, VEC>(a.x_out + base + c, x[i]);
+    if (a.h != nullptr && a.w_next == nullptr) store_t<T, VEC>(static_cast<T*>(a.h) + base + c, x[i]);
+  }
+  if (a.h == nullptr || a.w_next == nullptr) return;               // the same for every thread
+  const float rn = 1.0f / sqrtf(cta_sum(ss, s_part[1]) / (float)a.D + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= a.D) continue;
+    float g[VEC];
+    load_t<T, VEC>(static_cast<const T*>(a.w_next) + c, g);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) g[k] = x[i][k] * rn * (a.offset + g[k]);
+    store_t<T, VEC>(static_cast<T*>(a.h) + base + c, g);
+  }
+}
+
+// Groups per thread and threads of a row of D channels; 0 groups: the row is too wide.
+template <int VEC>
+inline int row_groups(int D, int* threads) {
+  const int g = (D + VEC - 1) / VEC;
+  const int nv = (g + kNormThreads - 1) / kNormThreads;
+  for (int n = 1; n <= 16; n *= 2)
+    if (nv <= n) {
+      *threads = min(kNormThreads, ((g + n - 1) / n + 31) / 32 * 32);
+      return n;
+    }
+  return 0;
+}
+
+// ---- relu(z + bias)^2 ---------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+bias_squared_relu_kernel(const T* z, int64_t z_rs, const T* __restrict__ bias, T* out, int64_t out_rs, int rows, int width) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * VEC;
+  if (c >= width) return;
+  float b[VEC] = {};
+  if (bias != nullptr) load_t<T, VEC>(bias + c, b);
+  // rows 4 at a time: their loads are in flight together
+  for (int64_t row = (int64_t)blockIdx.y * 4; row < rows; row += (int64_t)gridDim.y * 4) {
+    float f[4][VEC];
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+      if (row + r < rows) load_t<T, VEC>(z + (row + r) * z_rs + c, f[r]);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      if (row + r >= rows) continue;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) {
+        const float t = fmaxf(f[r][k] + b[k], 0.f);
+        f[r][k] = t * t;
+      }
+      store_t<T, VEC>(out + (row + r) * out_rs + c, f[r]);
+    }
+  }
+}
+
 // ---- gelu_tanh(gate) * up ---------------------------------------------------------------------------
 __device__ __forceinline__ float gelu_tanh(float z) {
   const float c = 0.7978845608028654f;                    // sqrt(2 / pi)
@@ -191,7 +376,72 @@ using namespace atma;
     else { using T = __nv_bfloat16; __VA_ARGS__; }                          \
   } while (0)
 
-extern "C" int atma_decoder_abi_version(void) { return 1; }
+#define ATMA_ROW_KERNEL(KERNEL, T, VEC, a)                                                                 \
+  do {                                                                                                     \
+    int threads = 0;                                                                                       \
+    const int nv = row_groups<VEC>(a.D, &threads);                                                         \
+    if (nv == 1) KERNEL<T, VEC, 1><<<rows, threads, 0, st>>>(a);                                           \
+    else if (nv == 2) KERNEL<T, VEC, 2><<<rows, threads, 0, st>>>(a);                                      \
+    else if (nv == 4) KERNEL<T, VEC, 4><<<rows, threads, 0, st>>>(a);                                      \
+    else if (nv == 8) KERNEL<T, VEC, 8><<<rows, threads, 0, st>>>(a);                                      \
+    else KERNEL<T, VEC, 16><<<rows, threads, 0, st>>>(a);                                                  \
+  } while (0)
+
+extern "C" int atma_decoder_abi_version(void) { return 2; }
+
+extern "C" int atma_embed_position_norm(const int32_t* ids, const int32_t* positions, const void* embed, const void* pos, const void* w,
+                                        float* x, void* h, int rows, int D, int vocab, int max_positions, float scale, float eps,
+                                        float offset, int dtype, void* stream) {
+  ATMA_REQUIRE(dtype == ATMA_F32 || dtype == ATMA_BF16, "embed_position_norm: unsupported dtype %d", dtype);
+  ATMA_REQUIRE(D > 0 && vocab > 0 && w != nullptr && x != nullptr, "embed_position_norm: bad arguments");
+  ATMA_REQUIRE(pos == nullptr || (positions != nullptr && max_positions > 0), "embed_position_norm: an empty position table");
+  if (rows <= 0) return ATMA_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int vb = dtype == ATMA_F32 ? 16 : 8;
+  const bool vec = D % 4 == 0 && aligned(x, 16) && aligned(embed, vb) && aligned(pos, vb) && aligned(w, vb) && aligned(h, vb);
+  ATMA_REQUIRE(D <= kNormThreads * 16 * (vec ? 4 : 1), "embed_position_norm: rows of %d channels", D);
+  const EmbedNormArgs a{ids, positions, embed, pos, w, x, h, D, vocab, max_positions, scale, eps, offset};
+  ATMA_DECODER_DISPATCH(dtype, T, {
+    if (vec) ATMA_ROW_KERNEL(embed_position_norm_kernel, T, 4, a);
+    else ATMA_ROW_KERNEL(embed_position_norm_kernel, T, 1, a);
+  });
+  return launch_status("embed_position_norm");
+}
+
+extern "C" int atma_residual_post_norm(const float* x, const void* y, const void* bias, const void* w, float* x_out, void* h,
+                                       const void* w_next, int rows, int D, float eps, float offset, int dtype, void* stream) {
+  ATMA_REQUIRE(dtype == ATMA_F32 || dtype == ATMA_BF16, "residual_post_norm: unsupported dtype %d", dtype);
+  ATMA_REQUIRE(D > 0 && x != nullptr && y != nullptr && w != nullptr, "residual_post_norm: bad arguments");
+  if (rows <= 0) return ATMA_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int vb = dtype == ATMA_F32 ? 16 : 8;
+  const bool vec = D % 4 == 0 && aligned(x, 16) && aligned(x_out, 16) && aligned(y, vb) && aligned(bias, vb) && aligned(w, vb) &&
+                   aligned(h, vb) && aligned(w_next, vb);
+  ATMA_REQUIRE(D <= kNormThreads * 16 * (vec ? 4 : 1), "residual_post_norm: rows of %d channels", D);
+  const PostNormArgs a{x, y, bias, w, x_out, h, w_next, D, eps, offset};
+  ATMA_DECODER_DISPATCH(dtype, T, {
+    if (vec) ATMA_ROW_KERNEL(residual_post_norm_kernel, T, 4, a);
+    else ATMA_ROW_KERNEL(residual_post_norm_kernel, T, 1, a);
+  });
+  return launch_status("residual_post_norm");
+}
+
+extern "C" int atma_bias_squared_relu(const void* z, int64_t z_rs, const void* bias, void* out, int64_t out_rs, int rows, int width,
+                                      int dtype, void* stream) {
+  ATMA_REQUIRE(dtype == ATMA_F32 || dtype == ATMA_BF16, "bias_squared_relu: unsupported dtype %d", dtype);
+  if (rows <= 0 || width <= 0) return ATMA_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  ATMA_DECODER_DISPATCH(dtype, T, {
+    constexpr int V = 16 / sizeof(T);
+    const bool vec = width % V == 0 && z_rs % V == 0 && out_rs % V == 0 && aligned(z, 16) && aligned(bias, 16) && aligned(out, 16);
+    const int per = 256 * (vec ? V : 1);
+    const dim3 grid((width + per - 1) / per, min((rows + 3) / 4, 65535));
+    const T *zp = (const T*)z, *bp = (const T*)bias;
+    if (vec) bias_squared_relu_kernel<T, V><<<grid, 256, 0, st>>>(zp, z_rs, bp, (T*)out, out_rs, rows, width);
+    else bias_squared_relu_kernel<T, 1><<<grid, 256, 0, st>>>(zp, z_rs, bp, (T*)out, out_rs, rows, width);
+  });
+  return launch_status("bias_squared_relu");
+}
 
 extern "C" int atma_embed_bigram(const int32_t* ids, const int32_t* prev, const void* embed, const void* bigram, float* x, int rows,
                                  int D, int vocab, int64_t mul_prev, int64_t mul_cur, int64_t buckets, int dtype, void* stream) {

@@ -1,6 +1,6 @@
 // Causal softmax attention over a paged cache, fp32 arithmetic throughout: the path for fp32 models and for head sizes
-// the tensor-core kernels do not serve, prompts and single tokens alike, with one or two maps per head and the
-// differential combination in the epilogue.  Also the entry points that choose between the kernels.
+// the tensor-core kernels do not serve, prompts and single tokens alike, with one or two maps per head, windows, a sink,
+// the differential combination and the output gate.  Also the entry points that choose between the kernels.
 //
 // A CTA of eight warps holds 16 query rows of one head, two per warp.  Keys come in tiles of 32: a lane owns a key for
 // the scores, and vdim / 32 value channels for the weighted sum, so the softmax statistics of a row are warp reductions.
@@ -42,6 +42,7 @@ softmax_rows_kernel(const atma_softmax_args a) {
   }
   const int last_pos = start + min(q0 + kTQ, n_rows) - 1;     // the last query's own position
   const int n_keys = min(last_pos + 1, a.max_blocks * a.block_size);
+  const KeyTiles tiles(start + q0, last_pos, a.max_blocks * a.block_size, a.window, a.keep_first, kTK);
   const int32_t* bt = a.block_tables + s * a.bt_stride;
 
   float m[kRPW][M], l[kRPW][M], acc[kRPW][M][NC];
@@ -49,12 +50,14 @@ softmax_rows_kernel(const atma_softmax_args a) {
   for (int r = 0; r < kRPW; ++r)
 #pragma unroll
     for (int t = 0; t < M; ++t) {
-      m[r][t] = -INFINITY; l[r][t] = 0.f;
+      m[r][t] = a.sink;                        // the sink is a key that was seen before the others
+      l[r][t] = a.sink > -INFINITY ? 1.f : 0.f;
 #pragma unroll
       for (int i = 0; i < NC; ++i) acc[r][t][i] = 0.f;
     }
 
-  for (int k0 = 0; k0 < n_keys; k0 += kTK) {
+  for (int kt = 0; kt < tiles.n; ++kt) {
+    const int k0 = tiles[kt] * kTK;
     __syncthreads();
     for (int j = warp; j < kTK; j += kWarps) {                // a warp per key row
       const int pos = k0 + j;
@@ -85,7 +88,7 @@ softmax_rows_kernel(const atma_softmax_args a) {
 #pragma unroll
       for (int r = 0; r < kRPW; ++r) {
         const int pos = start + q0 + warp * kRPW + r;
-        const float v = (k0 + lane <= pos && k0 + lane < n_keys) ? sc[r] : -INFINITY;
+        const float v = (k0 + lane < n_keys && key_visible(pos, k0 + lane, a.window, a.keep_first)) ? sc[r] : -INFINITY;
         const float mn = fmaxf(m[r][t], warp_max(v));
         const float p = mn == -INFINITY ? 0.f : expf(v - mn);
         const float al = mn == -INFINITY ? 1.f : expf(m[r][t] - mn);
@@ -117,8 +120,8 @@ softmax_rows_kernel(const atma_softmax_args a) {
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      o[i] = acc[r][0][i] / l[r][0];
-      if constexpr (M == 2) o[i] -= a.lambda * (acc[r][M - 1][i] / l[r][M - 1]);
+      o[i] = l[r][0] > 0.f ? acc[r][0][i] / l[r][0] : 0.f;
+      if constexpr (M == 2) o[i] -= l[r][M - 1] > 0.f ? a.lambda * (acc[r][M - 1][i] / l[r][M - 1]) : 0.f;
       ss = fmaf(o[i], o[i], ss);
     }
     float f = 1.f;
@@ -127,10 +130,11 @@ softmax_rows_kernel(const atma_softmax_args a) {
       f = a.out_scale / sqrtf(ss / (float)a.vdim + a.eps);
     }
     T* op = out + (int64_t)(r_begin + row) * a.out_rs + (int64_t)h * a.vdim;
+    const T* gp = a.gate == nullptr ? nullptr : static_cast<const T*>(a.gate) + (int64_t)(r_begin + row) * a.gate_rs + (int64_t)h * a.vdim;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
       const int c = lane + 32 * i;
-      if (c < a.vdim) op[c] = from_f32<T>(o[i] * f);
+      if (c < a.vdim) op[c] = from_f32<T>(o[i] * f * (gp != nullptr ? sigmoid_gate(gp[c]) : 1.f));
     }
   }
 }
@@ -173,6 +177,15 @@ int check(const atma_softmax_args* a, const char* what) {
   return ATMA_OK;
 }
 
+// Window and kept first keys within what index arithmetic on positions takes without overflow.
+atma_softmax_args bounded(const atma_softmax_args& a) {
+  constexpr int kMost = 1 << 30;
+  atma_softmax_args b = a;
+  b.window = min(max(a.window, 0), kMost);
+  b.keep_first = min(max(a.keep_first, 0), kMost);
+  return b;
+}
+
 int rows_path(const atma_softmax_args& a, int max_rows, cudaStream_t st) {
   return a.dtype == ATMA_F32 ? launch_rows_t<float>(a, max_rows, st) : launch_rows_t<__nv_bfloat16>(a, max_rows, st);
 }
@@ -189,8 +202,9 @@ extern "C" int atma_softmax_prefill(const atma_softmax_args* a, void* stream) {
   int rc = check(a, "softmax_prefill");
   if (rc != ATMA_OK) return rc;
   if (a->n_seqs <= 0 || a->max_rows <= 0) return ATMA_OK;
-  if (softmax_prefill_sm100_supported(*a)) return softmax_prefill_sm100(*a, (cudaStream_t)stream);
-  return rows_path(*a, a->max_rows, (cudaStream_t)stream);
+  const atma_softmax_args b = bounded(*a);
+  if (softmax_prefill_sm100_supported(b)) return softmax_prefill_sm100(b, (cudaStream_t)stream);
+  return rows_path(b, b.max_rows, (cudaStream_t)stream);
 }
 
 extern "C" int atma_softmax_decode(const atma_softmax_args* a, void* stream) {
@@ -199,9 +213,9 @@ extern "C" int atma_softmax_decode(const atma_softmax_args* a, void* stream) {
   if (a->n_seqs <= 0) return ATMA_OK;
   if (softmax_decode_mma_supported(*a)) {
     ATMA_REQUIRE(a->scratch != nullptr && a->n_splits > 0, "softmax_decode: scratch and n_splits are required");
-    return softmax_decode_mma(*a, (cudaStream_t)stream);
+    return softmax_decode_mma(bounded(*a), (cudaStream_t)stream);
   }
-  return rows_path(*a, 1, (cudaStream_t)stream);
+  return rows_path(bounded(*a), 1, (cudaStream_t)stream);
 }
 
 extern "C" int64_t atma_softmax_decode_scratch_floats(int n_seqs, int H, int maps, int vdim, int n_splits) {

@@ -1,5 +1,7 @@
 // Paged softmax attention of one query row per sequence, 16-bit caches: key ranges side by side, then a merge that also
-// applies the differential combination.
+// adds the sink to the denominator and applies the differential combination and the output gate.  With one map and a
+// single key range (short contexts and windows) the first kernel finishes by itself.  Key ranges are cut from the list of
+// key tiles that the row sees at all.
 //
 // A CTA streams the K and V rows of one key range of one (sequence, key/value head) through a cp.async ring of 64-key
 // tiles (16-byte copies, one page-table lookup per tile when tiles cannot straddle pages).  Keys are the rows of the
@@ -44,16 +46,27 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int gq = lane >> 2, tq = lane & 3;
 
-  const int n = max(0, min(a.start_pos[b] + 1, a.max_blocks * a.block_size));
-  int chunk = (n + a.n_splits - 1) / a.n_splits;
-  chunk = (chunk + kTileKeys - 1) / kTileKeys * kTileKeys;
-  const int lo = split * chunk, hi = min(lo + chunk, n);
+  const int pos = a.start_pos[b];
+  const int n = max(0, min(pos + 1, a.max_blocks * a.block_size));
+  const KeyTiles tiles(pos, pos, a.max_blocks * a.block_size, a.window, a.keep_first, kTileKeys);
+  const int per_split = (tiles.n + a.n_splits - 1) / a.n_splits;
+  const int tile0 = split * per_split, n_tiles = max(0, min(per_split, tiles.n - tile0));
+  const bool direct = MAPS == 1 && a.n_splits == 1;
   float* stats = a.scratch;                   // [b][h][map][split]{m, l}, then [b][h][map][split][VD]
   float* sacc = a.scratch + (int64_t)a.n_seqs * a.H * MAPS * a.n_splits * 2;
   auto part = [&](int col) {                  // column = map * GC + head
     return (((int64_t)b * a.H + h0 + col % GC) * MAPS + col / GC) * a.n_splits + split;
   };
-  if (lo >= hi) {                             // nothing in this range: weight zero in the merge
+  auto finish = [&](int c, int d, float v) {    // direct form: gate and store channel d of head h0 + c
+    const int64_t ch = (int64_t)(h0 + c) * VD + d;
+    if (a.gate != nullptr) v *= sigmoid_gate(static_cast<const __nv_bfloat16*>(a.gate)[b * a.gate_rs + ch]);
+    static_cast<__nv_bfloat16*>(a.out)[b * a.out_rs + ch] = __float2bfloat16_rn(v);
+  };
+  if (n_tiles == 0) {                         // nothing in this range: weight zero in the merge
+    if (direct) {
+      for (int i = tid; i < nh * VD; i += 128) static_cast<__nv_bfloat16*>(a.out)[b * a.out_rs + (int64_t)h0 * VD + i] = __float2bfloat16_rn(0.f);
+      return;
+    }
     for (int c = warp; c < MAPS * GC; c += 4) {
       if (c % GC >= nh) continue;
       const int64_t p = part(c);
@@ -66,8 +79,7 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
   const uint16_t* V = static_cast<const uint16_t*>(a.v_cache) + (int64_t)g * VD;
   const int64_t krow = (int64_t)a.G * KD, vrow = (int64_t)a.G * VD;
   const int32_t* bt = a.block_tables + b * a.bt_stride;
-  const int n_tiles = (hi - lo + kTileKeys - 1) / kTileKeys;
-  const bool tile_in_page = a.block_size % kTileKeys == 0;       // lo is a multiple of the tile
+  const bool tile_in_page = a.block_size % kTileKeys == 0;
 
   auto row_of = [&](int pos) {
     const int blk = pos / a.block_size;
@@ -75,19 +87,19 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
   };
   auto load_tile = [&](int it) {
     const uint32_t dst = smem_u32(sm + (it % STAGES) * kStage);
-    const int pos0 = lo + it * kTileKeys;
+    const int pos0 = tiles[tile0 + it] * kTileKeys;
     const int64_t base = tile_in_page ? row_of(pos0) : 0;
 #pragma unroll
     for (int j = 0; j < kTileKeys * CK / 128; ++j) {
       const int i = tid + j * 128, r = i / CK, ch = i % CK;
-      const bool ok = pos0 + r < hi;
+      const bool ok = pos0 + r < n && key_visible(pos, pos0 + r, a.window, a.keep_first);
       const int64_t row = !ok ? 0 : (tile_in_page ? base + r : row_of(pos0 + r));
       cp_async16(dst + tile_off(r, ch * 8, KD), K + row * krow + ch * 8, ok);
     }
 #pragma unroll
     for (int j = 0; j < kTileKeys * CV / 128; ++j) {
       const int i = tid + j * 128, r = i / CV, ch = i % CV;
-      const bool ok = pos0 + r < hi;
+      const bool ok = pos0 + r < n && key_visible(pos, pos0 + r, a.window, a.keep_first);
       const int64_t row = !ok ? 0 : (tile_in_page ? base + r : row_of(pos0 + r));
       cp_async16(dst + kKBytes + tile_off(r, ch * 8, VD), V + row * vrow + ch * 8, ok);
     }
@@ -139,8 +151,9 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) S[e] += S2[e];
-    const int key0 = lo + it * kTileKeys + 16 * warp + gq;
-    const bool ok0 = key0 < hi, ok1 = key0 + 8 < hi;
+    const int key0 = tiles[tile0 + it] * kTileKeys + 16 * warp + gq;
+    const bool ok0 = key0 < n && key_visible(pos, key0, a.window, a.keep_first);
+    const bool ok1 = key0 + 8 < n && key_visible(pos, key0 + 8, a.window, a.keep_first);
     float x[4];                               // [key gq][e], [key gq + 8][e]
     x[0] = ok0 ? S[0] * sc : -INFINITY; x[1] = ok0 ? S[1] * sc : -INFINITY;
     x[2] = ok1 ? S[2] * sc : -INFINITY; x[3] = ok1 ? S[3] * sc : -INFINITY;
@@ -206,6 +219,17 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     }
   }
   __syncthreads();
+  if (direct) {
+    for (int i = tid; i < nh * VD; i += 128) {
+      const int c = i / VD, d = i - c * VD;
+      const float M = fmaxf(fmaxf(s_m[c], s_m[8 + c]), fmaxf(s_m[16 + c], s_m[24 + c])), s2 = a.sink * kLog2e;
+      const float M2 = fmaxf(M, s2), w = exp2f(M - M2);
+      const float l = (s_l[c] + s_l[8 + c] + s_l[16 + c] + s_l[24 + c]) * w + exp2f(s2 - M2);
+      const float acc = (s_o[c * OLD + d] + s_o[(8 + c) * OLD + d] + s_o[(16 + c) * OLD + d] + s_o[(24 + c) * OLD + d]) * w;
+      finish(c, d, l > 0.f ? acc / l : 0.f);
+    }
+    return;
+  }
   for (int i = tid; i < MAPS * GC * VD; i += 128) {
     const int c = i / VD, d = i - c * VD;
     if (c % GC >= nh) continue;
@@ -233,15 +257,16 @@ softmax_decode_merge_kernel(const atma_softmax_args a) {
 #pragma unroll
   for (int m = 0; m < MAPS; ++m) {
     const int64_t p0 = (((int64_t)b * a.H + h) * MAPS + m) * a.n_splits;
-    float M = kNegBig;
+    const float s2 = a.sink * kLog2e;
+    float M = fmaxf(kNegBig, s2);
     for (int s = 0; s < a.n_splits; ++s) M = fmaxf(M, stats[2 * (p0 + s)]);
-    float l = 0.f, acc = 0.f;
+    float l = exp2f(s2 - M), acc = 0.f;
     for (int s = 0; s < a.n_splits; ++s) {
       const float w = exp2f(stats[2 * (p0 + s)] - M);
       l = fmaf(stats[2 * (p0 + s) + 1], w, l);
       acc = fmaf(sacc[(p0 + s) * VD + d], w, acc);
     }
-    o[m] = acc / l;
+    o[m] = l > 0.f ? acc / l : 0.f;
   }
   float v = o[0];
   if constexpr (MAPS == 2) {
@@ -254,6 +279,7 @@ softmax_decode_merge_kernel(const atma_softmax_args a) {
     for (int i = 0; i < VD / 32; ++i) ss += s_part[i];
     v *= a.out_scale / sqrtf(ss / (float)VD + a.eps);
   }
+  if (a.gate != nullptr) v *= sigmoid_gate(static_cast<const __nv_bfloat16*>(a.gate)[b * a.gate_rs + (int64_t)h * VD + d]);
   *out = __float2bfloat16_rn(v);
 }
 
@@ -268,7 +294,7 @@ int launch(const atma_softmax_args& a, cudaStream_t st) {
   auto kern = softmax_decode_split_kernel<MAPS, DIM, VD, kStages>;
   ATMA_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   kern<<<dim3(a.n_splits, a.G * ((rep + GC - 1) / GC), a.n_seqs), 128, smem, st>>>(a);
-  softmax_decode_merge_kernel<MAPS, VD><<<dim3(a.H, a.n_seqs), VD, 0, st>>>(a);
+  if (MAPS == 2 || a.n_splits > 1) softmax_decode_merge_kernel<MAPS, VD><<<dim3(a.H, a.n_seqs), VD, 0, st>>>(a);
   return launch_status("softmax_decode (mma)");
 }
 

@@ -1,22 +1,25 @@
-// Differential softmax attention of prompt rows on the 5th-generation tensor cores (sm_100a), keys and values read from
-// the paged cache by TMA.
+// Softmax attention of prompt rows on the 5th-generation tensor cores (sm_100a), keys and values read from the paged
+// cache by TMA; one map per head, or two with the differential combination.
 //
-// One CTA owns a 128-row query tile of one head, both maps: S_m = Q_m K_m^T (SS) and O_m += P_m V (P from TMEM) for
-// m = 0, 1.  The maps ping-pong on the tensor pipe - while the softmax warps of one work on their scores the other's
-// products run - and every V tile brought into shared memory feeds both.  A 128-key tile lies inside one page (the page
-// size is a multiple of 128), so the producer turns a key tile into a cache row with one page-table lookup.
+// One CTA owns a 128-row query tile and two streams m = 0, 1 over its keys, S_m = Q_m K_m^T (SS) and O_m += P_m V_m (P
+// from TMEM).  The streams ping-pong on the tensor pipe: while the softmax warps of one work on their scores the other's
+// products run.  With two maps the streams are the maps of one head (K tiles apart, V tiles shared); with one map they are
+// two neighbouring query heads, which share K and V tiles where they belong to the same key/value head (an odd last head
+// runs alone).  A 128-key tile lies inside one page (the page size is a multiple of 128), so the producer turns a key tile
+// into a cache row with one page-table lookup.  Key tiles that no row of the tile sees are left out.
 //
-//   warp 0      TMA producer: both Q tiles once, K tiles (map 0, map 1, map 0, ...) and V tiles through rings
+//   warp 0      TMA producer: the Q tiles once, K and V tiles (stream 0, stream 1, stream 0, ... or shared) through rings
 //   warp 1      MMA issuer (one lane)
 //   warps 2-3   idle (they complete the first warpgroup, whose registers are handed over)
-//   warps 4-7   softmax of map 0, one thread per query row (= one TMEM lane); half of the epilogue's channels
-//   warps 8-11  softmax of map 1; the other half
+//   warps 4-7   softmax of stream 0, one thread per query row (= one TMEM lane), and its epilogue (two maps: half of the
+//               epilogue's channels)
+//   warps 8-11  softmax of stream 1; its epilogue or the other half
 // TMEM (512 columns): S_0 [0,128) S_1 [128,256) O_0 [256,384) O_1 [384,512).  P_m overwrites S_m once the row is in
 // registers, as two 16-bit terms - the rounded weight in the first 64 columns, the remainder in the second - so that the
 // weights enter the product with 16 bits of mantissa; O_m += P_hi V + P_lo V.
-// Rows stream (m, L = sum p, O = sum p v) in the log2 domain; the maximum in use moves only when it grew by more than
-// 2^8.  The epilogue forms o = O_0/L_0 - lambda O_1/L_1 over half of the channels per warpgroup, exchanges the sums of
-// squares and writes o * out_scale / rms(o).
+// Rows stream (m, L = sum p, O = sum p v) in the log2 domain, starting from the sink (its score, 1, 0) if there is one; the
+// maximum in use moves only when it grew by more than 2^8.  With two maps the epilogue forms o = O_0/L_0 - lambda O_1/L_1 over half of the channels per warpgroup, exchanges the sums of
+// squares and writes o * out_scale / rms(o); with one map it writes O/L.  Both apply the output gate.
 // Every mbarrier wait is bounded; on expiry the CTA frees its TMEM, returns and leaves a status word for the host.
 #include "softmax_attention.cuh"
 #include "sm100.cuh"
@@ -63,7 +66,7 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
 }
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int DIM, int VD>
+template <int MAPS, int DIM, int VD>
 __global__ void __launch_bounds__(kThreads, 1)
 softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                              const __grid_constant__ CUtensorMap tmap_v, const atma_softmax_args a) {
@@ -82,12 +85,15 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
   float (*s_ss)[kBM] = s_l + 2;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int seq = a.tile_seq[blockIdx.x], row0 = a.tile_row[blockIdx.x], h = blockIdx.y, g = h / (a.H / a.G);
+  const int seq = a.tile_seq[blockIdx.x], row0 = a.tile_row[blockIdx.x];
+  // head and key/value head of each stream; K and V tiles per key tile
+  const int h0 = MAPS == 2 ? blockIdx.y : 2 * blockIdx.y, h1 = MAPS == 2 ? h0 : h0 + 1;
+  const int n_streams = h1 < a.H ? 2 : 1;
+  const int g0 = h0 / (a.H / a.G), g1 = min(h1, a.H - 1) / (a.H / a.G);
+  const int nv = g0 == g1 ? 1 : 2, nk = MAPS == 2 ? 2 : nv;
   const int r_begin = a.cu_rows[seq], n_rows = a.cu_rows[seq + 1] - r_begin, start = a.start_pos[seq];
-  // key tiles of this query tile: up to its last row's own position
-  int n_kt = (start + min(row0 + kBM, n_rows) - 1) / kBN + 1;
-  n_kt = min(n_kt, a.max_blocks * (a.block_size / kBN));
-  if (start < 0 || row0 >= n_rows) n_kt = 0;
+  const KeyTiles tiles(start + row0, start + min(row0 + kBM, n_rows) - 1, a.max_blocks * a.block_size, a.window, a.keep_first, kBN);
+  const int n_kt = start < 0 || row0 >= n_rows ? 0 : tiles.n;
 
   if (tid == 0) {
     for (int i = 0; i < 2; ++i) {
@@ -118,35 +124,35 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
       // ============================= TMA producer ==============================================
       if (lane == 0 && n_kt > 0) {
         const int32_t* bt = a.block_tables + seq * a.bt_stride;
-#pragma unroll
-        for (int m = 0; m < 2; ++m) {
+        for (int m = 0; m < n_streams; ++m) {
           mbar_arrive_expect_tx(&bar.q_full[m], kMapTile);
 #pragma unroll
           for (int cb = 0; cb < DIM / 64; ++cb)
-            tma_load_4d(sQ + m * kMapTile + cb * kBox, &tmap_q, &bar.q_full[m], (h * 2 + m) * DIM + cb * 64, r_begin + row0, 0, 0);
+            tma_load_4d(sQ + m * kMapTile + cb * kBox, &tmap_q, &bar.q_full[m], (MAPS == 2 ? h0 * 2 + m : h0 + m) * DIM + cb * 64,
+                        r_begin + row0, 0, 0);
         }
         bool ok = true;
         for (int j = 0; j < n_kt && ok; ++j) {
-          const int blk = j * kBN / a.block_size;
-          const int row = min(max(bt[blk], 0), a.num_blocks - 1) * a.block_size + (j * kBN - blk * a.block_size);
-#pragma unroll
-          for (int m = 0; m < 2; ++m) {
-            const int i = 2 * j + m, s = i % KS;
+          const int key0 = tiles[j] * kBN, blk = key0 / a.block_size;
+          const int row = min(max(bt[blk], 0), a.num_blocks - 1) * a.block_size + (key0 - blk * a.block_size);
+          for (int m = 0; m < nk; ++m) {
+            const int i = nk * j + m, s = i % KS;
             ok = ok && mbar_wait(&bar.k_empty[s], ((uint32_t)(i / KS) & 1u) ^ 1u, abort_flag);
             if (!ok) break;
             mbar_arrive_expect_tx(&bar.k_full[s], kMapTile);
 #pragma unroll
             for (int cb = 0; cb < DIM / 64; ++cb)
-              tma_load_4d(sK + s * kMapTile + cb * kBox, &tmap_k, &bar.k_full[s], (g * 2 + m) * DIM + cb * 64, row, 0, 0);
+              tma_load_4d(sK + s * kMapTile + cb * kBox, &tmap_k, &bar.k_full[s], (MAPS == 2 ? g0 * 2 + m : (m == 0 ? g0 : g1)) * DIM + cb * 64, row, 0, 0);
           }
-          if (!ok) break;
-          const int s = j % kVStages;
-          ok = mbar_wait(&bar.v_empty[s], ((uint32_t)(j / kVStages) & 1u) ^ 1u, abort_flag);
-          if (!ok) break;
-          mbar_arrive_expect_tx(&bar.v_full[s], kVTile);
+          for (int m = 0; m < nv && ok; ++m) {
+            const int i = nv * j + m, s = i % kVStages;
+            ok = mbar_wait(&bar.v_empty[s], ((uint32_t)(i / kVStages) & 1u) ^ 1u, abort_flag);
+            if (!ok) break;
+            mbar_arrive_expect_tx(&bar.v_full[s], kVTile);
 #pragma unroll
-          for (int cb = 0; cb < VD / 64; ++cb)
-            tma_load_4d(sV + s * kVTile + cb * kBox, &tmap_v, &bar.v_full[s], g * VD + cb * 64, row, 0, 0);
+            for (int cb = 0; cb < VD / 64; ++cb)
+              tma_load_4d(sV + s * kVTile + cb * kBox, &tmap_v, &bar.v_full[s], (m == 0 ? g0 : g1) * VD + cb * 64, row, 0, 0);
+          }
         }
       }
       __syncwarp();
@@ -177,38 +183,32 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
               mma_ts(od, pa + half * 64 + kk * 8, b0 + uint64_t(kk * (2048 >> 4)), idesc_pv, (half > 0 || kk > 0 || acc) ? 1u : 0u);
         };
         bool ok = true;
-#pragma unroll
-        for (int m = 0; m < 2; ++m) {
-          ok = ok && mbar_wait(&bar.q_full[m], 0, abort_flag) && mbar_wait(&bar.k_full[m], 0, abort_flag);
-          if (ok) {
-            tc_fence_after();
-            issue_qk(m, m);
-            tc_commit(&bar.s_full[m]);
-            tc_commit(&bar.k_empty[m]);
-          }
-        }
+        // a tile that both streams read is given back by the last of them
+        const int last = n_streams - 1;
+        auto next_qk = [&](int m, int j) {
+          const int i = nk == 2 ? 2 * j + m : j, s = i % KS;
+          if (!mbar_wait(&bar.k_full[s], (uint32_t)(i / KS) & 1u, abort_flag)) return false;
+          tc_fence_after();
+          issue_qk(m, s);
+          tc_commit(&bar.s_full[m]);
+          if (nk == 2 || m == last) tc_commit(&bar.k_empty[s]);
+          return true;
+        };
+        for (int m = 0; m < n_streams && ok; ++m) ok = mbar_wait(&bar.q_full[m], 0, abort_flag) && next_qk(m, 0);
         for (int j = 0; j < n_kt && ok; ++j) {
-          const int vs = j % kVStages;
           const bool more = j + 1 < n_kt;
 #pragma unroll
           for (int m = 0; m < 2; ++m) {
-            if (ok) ok = mbar_wait(&bar.p_full[m], (uint32_t)j & 1u, abort_flag);
-            if (ok && m == 0) ok = mbar_wait(&bar.v_full[vs], (uint32_t)(j / kVStages) & 1u, abort_flag);
+            if (!ok || m >= n_streams) break;
+            const int i = nv == 2 ? 2 * j + m : j, vs = i % kVStages;
+            ok = mbar_wait(&bar.p_full[m], (uint32_t)j & 1u, abort_flag) && mbar_wait(&bar.v_full[vs], (uint32_t)(i / kVStages) & 1u, abort_flag);
             if (!ok) break;
             tc_fence_after();
             issue_pv(m, vs, j > 0);
-            if (!more) tc_commit(&bar.o_final[m]);
-            if (more) {
-              const int i = 2 * (j + 1) + m, s = i % KS;
-              ok = mbar_wait(&bar.k_full[s], (uint32_t)(i / KS) & 1u, abort_flag);
-              if (!ok) break;
-              tc_fence_after();
-              issue_qk(m, s);
-              tc_commit(&bar.s_full[m]);
-              tc_commit(&bar.k_empty[s]);
-            }
+            if (nv == 2 || m == last) tc_commit(&bar.v_empty[vs]);
+            if (more) ok = next_qk(m, j + 1);
+            else tc_commit(&bar.o_final[m]);
           }
-          if (ok) tc_commit(&bar.v_empty[vs]);
         }
       }
       __syncwarp();
@@ -223,14 +223,18 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
     const uint32_t lane_base = tbase + (uint32_t(32 * (warp & 3)) << 16);
     const uint32_t tS = lane_base + m * 128, tO = lane_base + 256 + m * 128;
     const float sc2 = a.scale * kLog2e;
-    float m_used = kNegInit, m_run = kNegInit, L = 0.f;
+    const bool sink = a.sink > -INFINITY;
+    float m_used = sink ? a.sink * kLog2e : kNegInit, m_run = m_used, L = sink ? 1.f : 0.f;
     bool ok = true;
-    for (int j = 0; j < n_kt; ++j) {
+    const int my_tiles = m < n_streams ? n_kt : 0;
+    for (int j = 0; j < my_tiles; ++j) {
       ok = mbar_wait(&bar.s_full[m], (uint32_t)j & 1u, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int vis = row_ok ? pos + 1 - j * kBN : 0;             // key columns below this one are seen
+      const int key0 = tiles[j] * kBN;
+      const int vis = row_ok ? pos + 1 - key0 : 0;                // key columns from win (or below kept) to vis are seen
+      const int win = pos - a.window + 1 - key0, kept = a.keep_first - key0;
       uint32_t s[kBN];
 #pragma unroll
       for (int ch = 0; ch < 4; ++ch) tmem_ld32_nowait(tS + ch * 32, &s[ch * 32]);
@@ -241,6 +245,11 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
 #pragma unroll
         for (int i = 0; i < kBN; ++i)
           if (i >= vis) s[i] = 0xff800000u;                       // -inf
+      }
+      if (win > 0 && kept < kBN) {
+#pragma unroll
+        for (int i = 0; i < kBN; ++i)
+          if (i < win && i >= kept) s[i] = 0xff800000u;
       }
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
 #pragma unroll
@@ -293,48 +302,96 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
       __syncwarp();
       if (lane == 0) mbar_arrive(&bar.p_full[m]);
     }
-    // ---- epilogue: both maps' accumulators, half of the channels per warpgroup.  The barriers are met on every path. ----
-    if (ok && n_kt > 0) {
-      ok = mbar_wait(&bar.o_final[0], 0, abort_flag) && mbar_wait(&bar.o_final[1], 0, abort_flag);
-      ok = __all_sync(0xffffffffu, ok);
-      tc_fence_after();
-    }
-    s_l[m][r] = L;
-    softmax_sync();
-    const bool live = ok && n_kt > 0;
-    const float i0 = 1.0f / s_l[0][r], i1 = a.lambda / s_l[1][r];
-    constexpr int HC = VD / 2;
-    float o[HC];
-    float ss = 0.f;
-#pragma unroll
-    for (int ch = 0; ch < HC / 32; ++ch) {
-      uint32_t u0[32], u1[32];
-      if (live) {
-        tmem_ld32(lane_base + 256 + m * HC + ch * 32, u0);
-        tmem_ld32(lane_base + 384 + m * HC + ch * 32, u1);
-      } else {
-#pragma unroll
-        for (int i = 0; i < 32; ++i) u0[i] = u1[i] = 0u;
+    // ---- epilogue ----
+    if constexpr (MAPS == 1) {                                    // each warpgroup its own head
+      if (ok && my_tiles > 0) {
+        ok = __all_sync(0xffffffffu, mbar_wait(&bar.o_final[m], 0, abort_flag));
+        tc_fence_after();
       }
+      const bool live = ok && my_tiles > 0;
+      if (m < n_streams) {
+        const float inv = L > 0.f ? 1.0f / L : 0.f;
+        const int64_t row = r_begin + row0 + r;
+        __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + row * a.out_rs + (int64_t)(h0 + m) * VD;
+        const __nv_bfloat16* gp = static_cast<const __nv_bfloat16*>(a.gate) + row * a.gate_rs + (int64_t)(h0 + m) * VD;
+#pragma unroll 1
+        for (int ch = 0; ch < VD; ch += 32) {
+          uint32_t u[32];
+          if (live) {
+            tmem_ld32(tO + ch, u);
+          } else {
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        o[ch * 32 + i] = __uint_as_float(u0[i]) * i0 - __uint_as_float(u1[i]) * i1;
-        ss = fmaf(o[ch * 32 + i], o[ch * 32 + i], ss);
-      }
-    }
-    s_ss[m][r] = ss;
-    softmax_sync();
-    const float f = a.out_scale / sqrtf((s_ss[0][r] + s_ss[1][r]) / (float)VD + a.eps);
-    if (row_ok) {
-      __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + (int64_t)(r_begin + row0 + r) * a.out_rs + (int64_t)h * VD + m * HC;
+            for (int i = 0; i < 32; ++i) u[i] = 0u;
+          }
 #pragma unroll
-      for (int i = 0; i < HC; i += 8) {
-        uint4 w = make_uint4(0u, 0u, 0u, 0u);
-        if (live) {
-          w = make_uint4(pack_bf16(o[i] * f, o[i + 1] * f), pack_bf16(o[i + 2] * f, o[i + 3] * f), pack_bf16(o[i + 4] * f, o[i + 5] * f),
-                         pack_bf16(o[i + 6] * f, o[i + 7] * f));
+          for (int i = 0; i < 32; i += 8) {
+            if (!row_ok) break;
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(u[i + e]) * inv;
+            if (a.gate != nullptr) {
+              const uint4 z = *reinterpret_cast<const uint4*>(gp + ch + i);
+              const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                o[2 * e] *= 1.0f / (1.0f + __expf(-__uint_as_float(zw[e] << 16)));
+                o[2 * e + 1] *= 1.0f / (1.0f + __expf(-__uint_as_float(zw[e] & 0xffff0000u)));
+              }
+            }
+            *reinterpret_cast<uint4*>(op + ch + i) = make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]), pack_bf16(o[6], o[7]));
+          }
+          __syncwarp();
         }
-        *reinterpret_cast<uint4*>(op + i) = w;
+      }
+    } else {                  // both maps' accumulators, half of the channels per warpgroup; the barriers are met on every path
+      if (ok && n_kt > 0) {
+        ok = mbar_wait(&bar.o_final[0], 0, abort_flag) && mbar_wait(&bar.o_final[1], 0, abort_flag);
+        ok = __all_sync(0xffffffffu, ok);
+        tc_fence_after();
+      }
+      s_l[m][r] = L;
+      softmax_sync();
+      const bool live = ok && n_kt > 0;
+      const float i0 = s_l[0][r] > 0.f ? 1.0f / s_l[0][r] : 0.f, i1 = s_l[1][r] > 0.f ? a.lambda / s_l[1][r] : 0.f;
+      constexpr int HC = VD / 2;
+      float o[HC];
+      float ss = 0.f;
+#pragma unroll
+      for (int ch = 0; ch < HC / 32; ++ch) {
+        uint32_t u0[32], u1[32];
+        if (live) {
+          tmem_ld32(lane_base + 256 + m * HC + ch * 32, u0);
+          tmem_ld32(lane_base + 384 + m * HC + ch * 32, u1);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) u0[i] = u1[i] = 0u;
+        }
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          o[ch * 32 + i] = __uint_as_float(u0[i]) * i0 - __uint_as_float(u1[i]) * i1;
+          ss = fmaf(o[ch * 32 + i], o[ch * 32 + i], ss);
+        }
+      }
+      s_ss[m][r] = ss;
+      softmax_sync();
+      const float f = a.out_scale / sqrtf((s_ss[0][r] + s_ss[1][r]) / (float)VD + a.eps);
+      if (row_ok) {
+        const int64_t row = r_begin + row0 + r, ch0 = (int64_t)h0 * VD + m * HC;
+        __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + row * a.out_rs + ch0;
+        if (a.gate != nullptr) {
+          const __nv_bfloat16* gp = static_cast<const __nv_bfloat16*>(a.gate) + row * a.gate_rs + ch0;
+#pragma unroll
+          for (int i = 0; i < HC; ++i) o[i] *= sigmoid_gate(gp[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < HC; i += 8) {
+          uint4 w = make_uint4(0u, 0u, 0u, 0u);
+          if (live) {
+            w = make_uint4(pack_bf16(o[i] * f, o[i + 1] * f), pack_bf16(o[i + 2] * f, o[i + 3] * f), pack_bf16(o[i + 4] * f, o[i + 5] * f),
+                           pack_bf16(o[i + 6] * f, o[i + 7] * f));
+          }
+          *reinterpret_cast<uint4*>(op + i) = w;
+        }
       }
     }
   }
@@ -351,18 +408,18 @@ int rows_map(CUtensorMap* out, const void* base, int64_t width, int64_t rows) {
   return make_tmap_16bit_4d(out, base, 1, dims, strides, box);
 }
 
-template <int DIM, int VD>
+template <int MAPS, int DIM, int VD>
 int launch(const atma_softmax_args& a, cudaStream_t st) {
   CUtensorMap mq, mk, mv;
   const int64_t slots = (int64_t)a.num_blocks * a.block_size;
-  int rc = rows_map(&mq, a.q, (int64_t)a.H * 2 * DIM, a.total_rows);
-  if (rc == ATMA_OK) rc = rows_map(&mk, a.k_cache, (int64_t)a.G * 2 * DIM, slots);
+  int rc = rows_map(&mq, a.q, (int64_t)a.H * MAPS * DIM, a.total_rows);
+  if (rc == ATMA_OK) rc = rows_map(&mk, a.k_cache, (int64_t)a.G * MAPS * DIM, slots);
   if (rc == ATMA_OK) rc = rows_map(&mv, a.v_cache, (int64_t)a.G * VD, slots);
   if (rc != ATMA_OK) return rc;
   constexpr int smem = (2 + Cfg<DIM>::kKSlots) * Cfg<DIM>::kMapTile + kVStages * kBN * VD * 2 + 1024;
-  auto kern = softmax_prefill_sm100_kernel<DIM, VD>;
+  auto kern = softmax_prefill_sm100_kernel<MAPS, DIM, VD>;
   ATMA_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  kern<<<dim3(a.n_tiles, a.H), kThreads, smem, st>>>(mq, mk, mv, a);
+  kern<<<dim3(a.n_tiles, MAPS == 2 ? a.H : (a.H + 1) / 2), kThreads, smem, st>>>(mq, mk, mv, a);
   return launch_status("softmax_prefill (tcgen05)");
 }
 
@@ -370,15 +427,19 @@ int launch(const atma_softmax_args& a, cudaStream_t st) {
 
 bool softmax_prefill_sm100_supported(const atma_softmax_args& a) {
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  return a.dtype == ATMA_BF16 && a.maps == 2 && (a.dim == 64 || a.dim == 128) && (a.vdim == 64 || a.vdim == 128) && a.block_size % kBN == 0 &&
-         a.scale >= 0.f && a.out_rs % 8 == 0 && al(a.q) && al(a.k_cache) && al(a.v_cache) && al(a.out) &&
+  return a.dtype == ATMA_BF16 && (a.maps == 1 || a.maps == 2) && (a.dim == 64 || a.dim == 128) && (a.vdim == 64 || a.vdim == 128) && a.block_size % kBN == 0 &&
+         a.scale >= 0.f && a.out_rs % 8 == 0 && al(a.q) && al(a.k_cache) && al(a.v_cache) && al(a.out) && a.gate_rs % 8 == 0 && al(a.gate) &&
          (int64_t)a.num_blocks * a.block_size < (int64_t(1) << 31);
 }
 
 int softmax_prefill_sm100(const atma_softmax_args& a, cudaStream_t st) {
   ATMA_REQUIRE(a.tile_seq != nullptr && a.tile_row != nullptr && a.n_tiles > 0, "softmax_prefill: the query tiles are required for this shape");
-  if (a.dim == 64) return a.vdim == 64 ? launch<64, 64>(a, st) : launch<64, 128>(a, st);
-  return a.vdim == 64 ? launch<128, 64>(a, st) : launch<128, 128>(a, st);
+  if (a.maps == 1) {
+    if (a.dim == 64) return a.vdim == 64 ? launch<1, 64, 64>(a, st) : launch<1, 64, 128>(a, st);
+    return a.vdim == 64 ? launch<1, 128, 64>(a, st) : launch<1, 128, 128>(a, st);
+  }
+  if (a.dim == 64) return a.vdim == 64 ? launch<2, 64, 64>(a, st) : launch<2, 64, 128>(a, st);
+  return a.vdim == 64 ? launch<2, 128, 64>(a, st) : launch<2, 128, 128>(a, st);
 }
 
 int softmax_sm100_status_fetch_and_clear(int* out) {

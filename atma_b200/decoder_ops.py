@@ -52,6 +52,44 @@ def residual_norms(x, y, weights, eps, offset=1.0, dtype=None, in_place=True):
     return hs
 
 
+def embed_position_norm(ids, positions, embed, pos, weight, eps, scale=1.0, offset=0.0):
+    """Rows s = embed[id] * scale + pos[position] (pos None = no second term), divided by their root mean square, times
+    (offset + weight).  Returns them in fp32 and in the tables' dtype (the same tensor for fp32)."""
+    _lib.require_cuda(embed, "embed_position_norm")
+    n, D = ids.numel(), embed.shape[1]
+    x = torch.empty((n, D), device=embed.device, dtype=torch.float32)
+    h = None if embed.dtype == torch.float32 else torch.empty((n, D), device=embed.device, dtype=embed.dtype)
+    _check(_lib.load_decoder().atma_embed_position_norm(_ptr(ids), _ptr(positions), _ptr(embed), _ptr(pos), _ptr(weight), _ptr(x), _ptr(h),
+                                                        n, D, embed.shape[0], 0 if pos is None else pos.shape[0], float(scale), float(eps),
+                                                        float(offset), _lib.dtype_code(embed), _lib.stream_ptr()))
+    return x, x if h is None else h
+
+
+def residual_post_norm(x, y, weight, eps, bias=None, next_weight=None, offset=0.0, in_place=True):
+    """Norm on a sublayer's output: t = y + bias; x (rows, D) fp32 becomes x + t / rms(t) * (offset + weight).  Returns
+    the new x in y's dtype (x itself for fp32) or, with ``next_weight``, its own norm times (offset + next_weight); not
+    ``in_place`` leaves x as it is."""
+    _lib.require_cuda(x, "residual_post_norm")
+    n, D = x.shape
+    if y.shape != x.shape or not y.is_contiguous() or not x.is_contiguous():
+        raise ValueError("x and y must be contiguous and of one shape")
+    h = None
+    if next_weight is not None or y.dtype != torch.float32 or not in_place:
+        h = torch.empty((n, D), device=x.device, dtype=y.dtype)
+    _check(_lib.load_decoder().atma_residual_post_norm(_ptr(x), _ptr(y), _ptr(bias), _ptr(weight), _ptr(x if in_place else None), _ptr(h),
+                                                       _ptr(next_weight), n, D, float(eps), float(offset), _lib.dtype_code(y),
+                                                       _lib.stream_ptr()))
+    return x if h is None else h
+
+
+def bias_squared_relu(z, bias, out):
+    """out = relu(z + bias)^2 (bias None = none; rows may be strided; out may be z)."""
+    _rows(z, "z"), _rows(out, "out")
+    _check(_lib.load_decoder().atma_bias_squared_relu(_ptr(z), z.stride(0), _ptr(bias), _ptr(out), out.stride(0), z.shape[0], z.shape[1],
+                                                      _lib.dtype_code(z), _lib.stream_ptr()))
+    return out
+
+
 def gelu_gate(gate, up, out):
     """out = gelu_tanh(gate) * up (rows may be strided)."""
     _rows(gate, "gate"), _rows(up, "up"), _rows(out, "out")
@@ -82,7 +120,27 @@ def rotary_store(z, positions, slot_mapping, table, k_cache, v_cache, *, heads, 
     return q
 
 
-def _softmax_args(q, k_cache, v_cache, group, out, scale, lam, out_scale, eps):
+def norm_store(z, slot_mapping, k_cache, v_cache, q_width, *, q_weight=None, k_weight=None, eps=0.0, v_first=None, lam=0.0):
+    """Of the projection rows z = [q | k | v | ...]: q and k divided by their root mean square over the whole projection,
+    times the weights (None = as they are); v or, with ``v_first``, (1 - lam) v + lam v_first.  k and v go to the cache
+    rows ``slot_mapping``; returns q (rows, q_width)."""
+    _lib.require_cuda(z, "norm_store")
+    _rows(z, "z")
+    n, nk, nv = z.shape[0], k_cache.shape[2] * k_cache.shape[3], v_cache.shape[2] * v_cache.shape[3]
+    if q_width + nk + nv > z.shape[1] or (v_first is not None and v_first.shape != (n, nv)):
+        raise ValueError("norm_store: z or v_first does not fit the cache")
+    q = torch.empty((n, q_width), device=z.device, dtype=z.dtype)
+    _check(_lib.load_decoder().atma_norm_store(_ptr(z), z.stride(0), _ptr(slot_mapping), _ptr(q_weight), _ptr(k_weight), _ptr(v_first),
+                                               0 if v_first is None else _rows(v_first, "v_first").stride(0), float(lam), float(eps),
+                                               _ptr(q), _ptr(k_cache), _ptr(v_cache), n, q_width, nk, nv, _lib.dtype_code(z),
+                                               _lib.stream_ptr()))
+    return q
+
+
+NO_WINDOW = 2 ** 31 - 1
+
+
+def _softmax_args(q, k_cache, v_cache, group, out, scale, lam=0.0, out_scale=1.0, eps=0.0, window=None, keep_first=0, sink=None, gate=None):
     n, H, maps, dim = q.shape
     _rows(out, "out")
     a = _lib.SoftmaxArgs()
@@ -94,14 +152,21 @@ def _softmax_args(q, k_cache, v_cache, group, out, scale, lam, out_scale, eps):
     a.num_blocks, a.block_size, a.G, a.vdim = k_cache.shape[0], k_cache.shape[1], v_cache.shape[2], v_cache.shape[3]
     a.H, a.maps, a.dim, a.dtype = H, maps, dim, _lib.dtype_code(q)
     a.scale, a.lambda_, a.out_scale, a.eps = float(scale), float(lam), float(out_scale), float(eps)
+    if gate is not None:
+        a.gate, a.gate_rs = gate.data_ptr(), _rows(gate, "gate").stride(0)
+    a.window, a.keep_first = NO_WINDOW if window is None else int(window), int(keep_first)
+    a.sink = float("-inf") if sink is None else float(sink)
     return a
 
 
-def softmax_prefill(q, k_cache, v_cache, group, out, *, scale, lam=0.0, out_scale=1.0, eps=0.0):
+def softmax_prefill(q, k_cache, v_cache, group, out, **options):
     """Causal softmax attention of a group's rows over the paged cache; with two maps the differential combination.
-    q (rows, H, maps, dim); caches (blocks, block_size, G, maps*dim | vdim); ``group``: an engine ``RowGroup``."""
+    q (rows, H, maps, dim); caches (blocks, block_size, G, maps*dim | vdim); ``group``: an engine ``RowGroup``.
+    Options: scale (needed); lam, out_scale, eps (two maps); window and keep_first (position i sees key j <= i if
+    i - j < window or j < keep_first; None = every key); sink (score of an added key without a value, None = none);
+    gate (rows, H*vdim): the result is multiplied by its sigmoid."""
     _lib.require_cuda(q, "softmax_prefill")
-    a = _softmax_args(q, k_cache, v_cache, group, out, scale, lam, out_scale, eps)
+    a = _softmax_args(q, k_cache, v_cache, group, out, **options)
     if group.tile_seq is not None:
         a.tile_seq, a.tile_row, a.n_tiles = group.tile_seq.data_ptr(), group.tile_row.data_ptr(), group.tile_seq.numel()
     _check(_lib.load_decoder().atma_softmax_prefill(ctypes.byref(a), _lib.stream_ptr()))
@@ -115,14 +180,15 @@ def decode_key_ranges(n_seqs, heads, kv_heads, maps, max_keys):
     return decode_num_splits(n_seqs, kv_heads * -(-(heads // kv_heads) // per_cta), max_keys, min_keys=256)
 
 
-def softmax_decode(q, k_cache, v_cache, group, out, *, scale, lam=0.0, out_scale=1.0, eps=0.0, n_splits=None):
+def softmax_decode(q, k_cache, v_cache, group, out, *, n_splits=None, **options):
     """The same for one row per sequence."""
     _lib.require_cuda(q, "softmax_decode")
     lib = _lib.load_decoder()
-    a = _softmax_args(q, k_cache, v_cache, group, out, scale, lam, out_scale, eps)
+    a = _softmax_args(q, k_cache, v_cache, group, out, **options)
     scratch = None
     if lib.atma_softmax_decode_path(ctypes.byref(a)):
-        a.n_splits = n_splits or decode_key_ranges(a.n_seqs, a.H, a.G, a.maps, a.max_blocks * a.block_size)
+        most = min(a.max_blocks * a.block_size, a.window + a.keep_first)
+        a.n_splits = n_splits or decode_key_ranges(a.n_seqs, a.H, a.G, a.maps, most)
         scratch = torch.empty(int(lib.atma_softmax_decode_scratch_floats(a.n_seqs, a.H, a.maps, a.vdim, a.n_splits)),
                               device=q.device, dtype=torch.float32)
         a.scratch = scratch.data_ptr()
@@ -216,6 +282,15 @@ def linear(x, weight, out=None):
     if out is None:
         return torch.mm(x, weight.t())
     return torch.mm(x, weight.t(), out=out)
+
+
+def squared_relu_linear(x, weight, bias=None):
+    """relu(x @ weight.T + bias)^2."""
+    from .inference_ops import decode_linear, decode_linear_supported
+    if decode_linear_supported(x, weight):
+        return decode_linear(x, weight, bias=bias, gated="plain_squared_relu", lib=_lib.load_decoder())
+    z = torch.mm(x, weight.t())
+    return bias_squared_relu(z, bias, z)
 
 
 def gelu_gated_linear(x, weight, out):

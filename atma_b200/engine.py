@@ -70,8 +70,10 @@ class Sequence:
     prompt_len: int = 0
     done: int = 0                     # tokens whose keys and state are in the cache
     slot: int = -1
-    pages: list = field(default_factory=list)
-    reserved: int = 0                 # pages promised at admission and not taken yet
+    pages: list = field(default_factory=list)     # page of every block of tokens, -1 = given back
+    dropped: int = 0                  # blocks below this one have been looked at for giving back
+    promised_blocks: int = 0          # blocks of tokens admitted for, 0 = no promise
+    reserved: int = 0                 # pages promised and not taken yet
     generator: torch.Generator = None
 
     @property
@@ -85,31 +87,59 @@ class OutOfCache(RuntimeError):
 
 class CacheManager:
     """Free lists of K/V pages and state slots.  Nothing is cleared on release: a sequence's first token starts its state
-    from zero and only keys at its own positions are read."""
+    from zero and only keys at its own positions are read.
 
-    def __init__(self, num_blocks, block_size, max_seqs, max_blocks_per_seq):
+    ``reach`` = (window, first): no layer looks back past a position's last ``window`` keys except at the first ``first``
+    ones, so a sequence gives back the pages in between as it grows and holds at most ``live_pages`` at a time when it
+    advances by up to ``max_portion`` tokens a step (None: every key stays)."""
+
+    def __init__(self, num_blocks, block_size, max_seqs, max_blocks_per_seq, reach=None, max_portion=None):
         self.num_blocks, self.block_size, self.max_seqs, self.max_blocks_per_seq = num_blocks, block_size, max_seqs, max_blocks_per_seq
+        self.reach, self.max_portion = reach, max_portion
         self.free_pages, self.free_slots = deque(range(num_blocks)), deque(range(max_seqs))
         self.promised = 0
 
     def pages_for(self, tokens):
         return -(-tokens // self.block_size)
 
+    def live_pages(self, total_tokens):
+        """The most pages that a sequence of ``total_tokens`` holds at any time."""
+        need = self.pages_for(total_tokens)
+        if self.reach is None or self.max_portion is None:
+            return need
+        window, first = self.reach
+        return min(need, self.pages_for(first) + self.pages_for(window + self.max_portion) + 1)
+
     def admit(self, seq, total_tokens=0):
         """A slot, and the promise of pages for ``total_tokens``; False if there is no room."""
-        need = self.pages_for(total_tokens)
-        if need > self.max_blocks_per_seq:
+        blocks, need = self.pages_for(total_tokens), self.live_pages(total_tokens)
+        if blocks > self.max_blocks_per_seq:
             raise ValueError(f"a sequence of {total_tokens} tokens exceeds the longest one this cache serves "
                              f"({self.max_blocks_per_seq * self.block_size})")
         if not self.free_slots or need > len(self.free_pages) - self.promised:
             return False
         seq.slot = self.free_slots.popleft()
-        seq.reserved = need
+        seq.promised_blocks, seq.reserved = blocks, need
         self.promised += need
         return True
 
+    def _drop_unseen(self, seq):
+        """Gives back the pages that no token after the first ``seq.done`` can see; what a promise still needs of them
+        stays promised."""
+        window, first = self.reach
+        keep, end = self.pages_for(first), max(seq.done + 1 - window, 0) // self.block_size       # blocks in [keep, end) are out of sight
+        for b in range(max(seq.dropped, keep), min(end, len(seq.pages))):
+            self.free_pages.append(seq.pages[b])
+            seq.pages[b] = -1
+            if seq.reserved < seq.promised_blocks - len(seq.pages):
+                seq.reserved += 1
+                self.promised += 1
+        seq.dropped = max(seq.dropped, end)
+
     def extend(self, seq, tokens):
-        """Pages for the sequence's first ``tokens`` tokens."""
+        """Pages for the sequence's first ``tokens`` tokens, of which ``seq.done`` are in the cache."""
+        if self.reach is not None:
+            self._drop_unseen(seq)
         need = self.pages_for(tokens)
         if need > self.max_blocks_per_seq:
             raise OutOfCache(f"a sequence of {tokens} tokens exceeds {self.max_blocks_per_seq * self.block_size}")
@@ -122,9 +152,9 @@ class CacheManager:
             seq.pages.append(self.free_pages.popleft())
 
     def release(self, seq):
-        self.free_pages.extend(seq.pages)
+        self.free_pages.extend(p for p in seq.pages if p >= 0)
         self.promised -= seq.reserved
-        seq.reserved = 0
+        seq.reserved = seq.promised_blocks = seq.dropped = 0
         if seq.slot >= 0:
             self.free_slots.append(seq.slot)
         seq.pages, seq.slot = [], -1
@@ -199,7 +229,7 @@ class ModelRunner:
         start = np.array([s.done for s, _ in plan], np.int64)
         tables = np.zeros((len(plan), width), np.int64)
         for i, (s, _) in enumerate(plan):
-            tables[i, :len(s.pages)] = s.pages
+            tables[i, :len(s.pages)] = s.pages                             # -1 where a page was given back: never read
         return lens, cu, start, tables
 
     def build(self, plan, want_rows, pad_decode_to=None):
@@ -359,15 +389,21 @@ def sample(logits, sequences):
 
 # ---- the engine --------------------------------------------------------------------------------------------------------
 class Engine:
-    """``max_tokens``: tokens that live sequences hold at most (sizes the K/V cache); ``max_model_len``: the longest
-    sequence (None = max_tokens)."""
+    """``max_tokens``: tokens whose keys live sequences hold at most (sizes the K/V cache); ``max_model_len``: the longest
+    sequence (None = max_tokens; more than that where the model only looks back a window)."""
 
     def __init__(self, model, *, max_tokens=32768, max_seqs=64, block_size=256, max_model_len=None, max_step_tokens=8192, graphs=True):
-        max_model_len = min(max_model_len or max_tokens, max_tokens)
+        reach, limit = getattr(model, "cache_reach", None), getattr(model, "max_positions", None)
+        max_model_len = max_model_len or max_tokens
+        if reach is None:
+            max_model_len = min(max_model_len, max_tokens)
+        if limit is not None:
+            max_model_len = min(max_model_len, limit)
         per_seq = -(-max_model_len // block_size)
+        self.max_len = per_seq * block_size if limit is None else min(per_seq * block_size, limit)
         num_blocks = -(-max_tokens // block_size) + max_seqs          # every live sequence may leave a page unfilled
         self.model = model
-        self.cache = CacheManager(num_blocks, block_size, max_seqs, per_seq)
+        self.cache = CacheManager(num_blocks, block_size, max_seqs, per_seq, reach, max_step_tokens)
         state = model.new_state(max_seqs, num_blocks, block_size, per_seq * block_size)
         self.runner = ModelRunner(model, self.cache, state, graphs)
         self.scheduler = Scheduler(self.cache, max_step_tokens, model.chunked_prefill, model.mixed_batches)
@@ -389,9 +425,8 @@ class Engine:
             raise ValueError("max_new_tokens must be at least 1")
         self._names += 1
         seq = Sequence(self._names, tokens, params, len(tokens))
-        limit = self.cache.max_blocks_per_seq * self.cache.block_size
-        if len(tokens) + params.max_new_tokens > limit:
-            raise ValueError(f"prompt and new tokens exceed the longest sequence served ({limit})")
+        if len(tokens) + params.max_new_tokens > self.max_len:
+            raise ValueError(f"prompt and new tokens exceed the longest sequence served ({self.max_len})")
         self.scheduler.add(seq)
         return seq
 
@@ -433,6 +468,8 @@ class Engine:
         for name, tokens, want in entries:
             self._check_ids(tokens)
             seq = self.fed.get(name)
+            if (len(seq.tokens) if seq else 0) + len(tokens) > self.max_len:
+                raise ValueError(f"sequence {name!r} exceeds the longest one served ({self.max_len})")
             if seq is None:
                 seq = Sequence(name, [])
                 if not self.cache.admit(seq):

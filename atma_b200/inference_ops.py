@@ -323,7 +323,8 @@ def decode_linear_supported(x, weight, gated=False):
             weight.is_contiguous() and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0)
 
 
-_GATES = {False: 0, None: 0, True: 1, "squared_relu": 1, "gelu_tanh": 2}
+_GATES = {False: 0, None: 0, True: 1, "squared_relu": 1, "gelu_tanh": 2, "plain_squared_relu": 3}
+_HALVES = (1, 2)                      # forms whose weight holds two projections
 
 
 @torch.no_grad()
@@ -332,6 +333,7 @@ def decode_linear(x, weight, bias=None, gated=False, out=None, lib=None):
     (``F.linear`` at these sizes).  ``gated``: the weight holds two projections (2F, K), first half and second half,
     and the result is (rows, F): True / "squared_relu" = second * relu(first)^2 - the fc GEMM and
     ``squared_relu_gate`` of inference/models/atma.py:87-97 in one launch -, "gelu_tanh" = gelu_tanh(first) * second.
+    "plain_squared_relu" has no second half: (rows, N) = relu(x @ weight.T + bias)^2.
     x (rows, K), weight (N, K) contiguous, 16-bit.  ``out``: where the result goes (contiguous rows, any row stride);
     ``lib``: the library to call (None = libatma_b200.so; libatma_decoder.so has the same entry)."""
     _lib.require_cuda(x, "decode_linear")
@@ -346,8 +348,8 @@ def decode_linear(x, weight, bias=None, gated=False, out=None, lib=None):
         bias = bias.to(x.dtype).contiguous()
     gate = _GATES[gated]
     if out is None:
-        out = torch.empty((B, N // 2 if gate else N), device=x.device, dtype=x.dtype)
-    elif out.shape != (B, N // 2 if gate else N) or out.dtype != x.dtype or out.stride(1) != 1:
+        out = torch.empty((B, N // 2 if gate in _HALVES else N), device=x.device, dtype=x.dtype)
+    elif out.shape != (B, N // 2 if gate in _HALVES else N) or out.dtype != x.dtype or out.stride(1) != 1:
         raise ValueError("out must have the result's shape and dtype and contiguous rows")
     _lib.check(lib.atma_decode_linear(_lib.ptr(x), x.stride(0), _lib.ptr(weight), _lib.ptr(bias), _lib.ptr(out), out.stride(0),
                                       B, N, K, gate, _lib.dtype_code(x), _lib.stream_ptr()), lib)

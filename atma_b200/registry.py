@@ -10,6 +10,10 @@ A registered class has
     mixed_batches           decoding sequences and prompt portions may share a step
     graph_decode            a step of decoding sequences only can be captured in a CUDA graph
     vocab
+and may have
+    max_positions           the longest sequence the design can represent (absent or None: no limit)
+    cache_reach             (window, first): later positions see only a sequence's last ``window`` and first ``first``
+                            keys, so that pages between them are given back (absent or None: every key stays)
 """
 
 import importlib
@@ -19,7 +23,8 @@ import torch
 
 from .checkpoint import read_config, read_safetensors
 
-_MODELS = {"Atma": ("atma_b200.model", "AtmaModel"), "Rizurax": ("atma_b200.rizurax", "RizuraxModel")}
+_MODELS = {"Atma": ("atma_b200.model", "AtmaModel"), "Rizurax": ("atma_b200.rizurax", "RizuraxModel"),
+           "Zemivik": ("atma_b200.zemivik", "ZemivikModel")}
 
 
 def architectures():

@@ -20,7 +20,8 @@ from types import SimpleNamespace
 import torch
 
 from . import decoder_ops as ops
-from .mixers import GatedDelta, RotaryTable, SoftmaxAttention
+from .configured import ConfiguredModel
+from .mixers import GatedDelta, SoftmaxAttention
 
 UNIT_EPS = 1e-6                # inside the root of the unit vectors of q and k
 
@@ -36,41 +37,18 @@ def layer_order(config):
     return list(range(start)) + list(range(start, stop)) * times + list(range(stop, n))
 
 
-class RizuraxModel:
-    kernel_library = "decoder"
-    chunked_prefill = mixed_batches = graph_decode = True
-
-    def __init__(self, config, tensors, dtype=torch.bfloat16, device="cuda"):
-        if dtype not in (torch.float32, torch.bfloat16):
-            raise ValueError(f"Rizurax runs in float32 or bfloat16, not {dtype}")
-        self.config, self.dtype, self.device = config, dtype, torch.device(device)
-        # matrix products accumulate in fp32 and are not split with 16-bit partial sums; fp32 means fp32
-        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        torch.backends.cuda.matmul.allow_tf32 = False
-        self.width, self.vocab, self.eps = config["width"], config["vocab"], float(config["norm"]["eps"])
+class RizuraxModel(ConfiguredModel):
+    def _build(self, config):
         self.order = layer_order(config)
-        self._tensors, self._tables = tensors, {}
         self.embed = self._w("embed", self.vocab, self.width)
         big = (config.get("embedding") or {}).get("bigram")
         self.bigram = self._w("bigram", big["buckets"] + 1, self.width) if big else None
         self.bigram_mul = (big["mul_prev"], big["mul_cur"]) if big else (0, 0)
         self.layers = [self._layer(i, e) for i, e in enumerate(config["layers"])]
         self.final_norm, self.head = self._w("final.norm", self.width), self._w("head", self.vocab, self.width)
-        del self._tensors
-
-    @classmethod
-    def from_config(cls, config, tensors, dtype=torch.bfloat16, device="cuda"):
-        return cls(config, tensors, dtype, device)
+        self.run_mixers = [self.layers[i].mixer for i in self.order]           # a looped layer has a cache per pass
 
     # ---- weights ----------------------------------------------------------------------------------------------
-    def _w(self, name, *shape, dtype=None):
-        if name not in self._tensors:
-            raise KeyError(f"the checkpoint has no tensor {name}")
-        t = self._tensors[name]
-        if shape and tuple(t.shape) != shape:
-            raise ValueError(f"tensor {name} is {tuple(t.shape)}, the configuration says {shape}")
-        return t.to(self.device, dtype or self.dtype).contiguous()
-
     def _layer(self, i, entry):
         p, D, m = f"l{i}.", self.width, entry["mixer"]
         kind = entry["type"]
@@ -101,13 +79,6 @@ class RizuraxModel:
                                 kv_heads=G, maps=2, dim=d, vdim=e, scale=float(m["scale"]), rotary=self._rotary(m.get("rot")), lam=lam,
                                 out_scale=1.0 - diff, eps=self.eps)
 
-    def _rotary(self, rot):
-        rot = rot or {"dims": 0, "base": 1.0}
-        key = repr(sorted((k, repr(v)) for k, v in rot.items()))
-        if key not in self._tables:
-            self._tables[key] = RotaryTable(rot["dims"], rot["base"], rot.get("scaling"), self.device)
-        return self._tables[key]
-
     def _delta(self, p, m):
         D, H, G, d, e, taps = self.width, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
         f32 = torch.float32
@@ -117,13 +88,7 @@ class RizuraxModel:
         return GatedDelta(self._w(p + "q", G * d, D), self._w(p + "k", G * d, D), self._w(p + "v", H * e, D), self._w(p + "g", H * e, D),
                           self._w(p + "a", H, D), self._w(p + "b", H, D), weights, self.eps)
 
-    # ---- state and step ---------------------------------------------------------------------------------------
-    def new_state(self, max_seqs, num_blocks, block_size=256, max_positions=None):
-        """One cache or state per layer run (a looped layer has one per pass)."""
-        for t in self._tables.values():
-            t.reserve(max_positions or num_blocks * block_size)
-        return [self.layers[i].mixer.new_state(max_seqs, num_blocks, block_size) for i in self.order]
-
+    # ---- the step ---------------------------------------------------------------------------------------------
     @torch.no_grad()
     def forward(self, batch, state, record=None):
         """One step: the batch's rows through all layers, caches and states updated; fp32 logits of ``batch.logit_rows``

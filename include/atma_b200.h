@@ -237,7 +237,8 @@ int atma_add_rms_norm(const void* x, const void* y, const void* weight, void* x_
  * (out has N/2 columns; bf16 rounds the square as eager execution does) - InferenceMLP.forward's
  * fc GEMM and squared_relu_gate in one launch (inference/models/atma.py:87-97); the plain form serves
  * its proj GEMM, the LFM2 in_proj / out_proj (:631-673) and the LM head at these batch sizes.
- * gated = 2: out[b][f] = gelu_tanh(first[f]) * second[f], the gated feed-forward of the decoder models.
+ * gated = 2: out[b][f] = gelu_tanh(first[f]) * second[f], the gated feed-forward of the decoder models; gated = 3: no
+ * second half, out[b][f] = relu(y[f])^2 for all N features.
  * K a multiple of 32, N of 16 (32 when gated); x rows 16-byte aligned. */
 int atma_decode_linear(const void* x, int64_t x_row_stride, const void* weight, const void* bias, void* out,
                        int64_t out_row_stride, int B, int N, int K, int gated, int dtype, void* stream);

@@ -1,8 +1,9 @@
 /*
  * atma_decoder - C ABI of the B200 (sm_100a) kernels for decoder-only language models that are assembled from a
- * configuration: softmax attention over a paged cache (one or two maps per head, rotary positions from a table),
- * the gated delta rule with per-head decay behind short convolutions, and the row operations around them (fp32
- * residual stream, zero-centred RMS norms, bigram embedding, gated feed-forward).
+ * configuration: softmax attention over a paged cache (one or two maps per head, rotary positions from a table or
+ * norms over the whole projections, sliding windows with kept first keys, a sink, an output gate), the gated delta
+ * rule with per-head decay behind short convolutions, and the row operations around them (fp32 residual stream, RMS
+ * norms in front of or behind a sublayer, bigram or learned-position embedding, feed-forward activations).
  *
  * Conventions as in atma_b200.h: plain device pointers, element strides, a CUDA stream passed as void*; nothing
  * allocates or synchronises; every call returns ATMA_OK or a negative atma_status and leaves a message for
@@ -34,6 +35,22 @@ int atma_embed_bigram(const int32_t* ids, const int32_t* prev, const void* embed
 int atma_residual_norms(const float* x, const void* y, float* x_out, const void* w1, void* h1, const void* w2, void* h2, int rows,
                         int D, float eps, float offset, int dtype, void* stream);
 
+/* s = embed[ids[row]] * scale + pos[positions[row]] (pos NULL = no second term); x = s / sqrt(mean s^2 + eps) *
+ * (offset + w), fp32 [rows][D]; h (NULL = not stored) receives x in the activation dtype. */
+int atma_embed_position_norm(const int32_t* ids, const int32_t* positions, const void* embed, const void* pos, const void* w, float* x,
+                             void* h, int rows, int D, int vocab, int max_positions, float scale, float eps, float offset, int dtype,
+                             void* stream);
+
+/* Norm on a sublayer's output: t = y + bias (bias NULL = none), x += t / sqrt(mean t^2 + eps) * (offset + w); x_out
+ * receives the sum (may equal x, NULL = not stored).  h (NULL = not stored) receives the sum in the activation dtype
+ * or, with w_next, the sum's own norm times (offset + w_next). */
+int atma_residual_post_norm(const float* x, const void* y, const void* bias, const void* w, float* x_out, void* h, const void* w_next,
+                            int rows, int D, float eps, float offset, int dtype, void* stream);
+
+/* out = relu(z + bias)^2 (bias NULL = none; out may be z), row strides in elements. */
+int atma_bias_squared_relu(const void* z, int64_t z_rs, const void* bias, void* out, int64_t out_rs, int rows, int width, int dtype,
+                           void* stream);
+
 /* out = gelu_tanh(gate) * up, row strides in elements. */
 int atma_gelu_gate(const void* gate, int64_t gate_rs, const void* up, int64_t up_rs, void* out, int64_t out_rs, int rows, int width,
                    int dtype, void* stream);
@@ -49,10 +66,21 @@ int atma_rotary_store(const void* z, int64_t z_rs, const int32_t* positions, con
                       int table_rows, void* q_out, void* k_cache, void* v_cache, int rows, int H, int G, int maps, int dim, int vdim,
                       int rot_dims, int dtype, void* stream);
 
+/* Norms over whole projections, value mixing and cache write in one pass.  z rows hold [q: q_width | k: k_width |
+ * v: v_width].  q / sqrt(mean q^2 + eps) * wq goes to q_out (dense), k / sqrt(mean k^2 + eps) * wk to row
+ * slot_mapping[row] of the k cache (wq, wk NULL = that part as it is), v or, with v_first,
+ * (1 - lambda) v + lambda v_first[row] to the same row of the v cache.  A negative slot is not stored. */
+int atma_norm_store(const void* z, int64_t z_rs, const int64_t* slot_mapping, const void* wq, const void* wk, const void* v_first,
+                    int64_t v_first_rs, float lambda, float eps, void* q_out, void* k_cache, void* v_cache, int rows, int q_width,
+                    int k_width, int v_width, int dtype, void* stream);
+
 /* Causal softmax attention of a step's rows over a paged cache that already holds their own keys.
  * q dense [rows][H][maps][dim]; k_cache [num_blocks*block_size][G][maps][dim]; v_cache [..][G][vdim]; query head h
  * reads key/value head h / (H/G).  maps = 1: out = attention.  maps = 2: both maps attend over the same values and
- * o = a1 - lambda * a2 is divided by its root mean square over vdim (eps inside the root) and multiplied by out_scale. */
+ * o = a1 - lambda * a2 is divided by its root mean square over vdim (eps inside the root) and multiplied by out_scale.
+ * Position i sees key j <= i if i - j < window (INT_MAX = every key) or j < keep_first.  sink: the score of an added
+ * key that has no value and only enters the denominator (-INFINITY = none).  gate [rows][H*vdim] (NULL = none): the
+ * result is multiplied by sigmoid(gate). */
 typedef struct {
   const void* q; const void* k_cache; const void* v_cache;
   const int32_t* block_tables; int64_t bt_stride;
@@ -67,6 +95,9 @@ typedef struct {
   int H, G, maps, dim, vdim;
   int num_blocks, block_size, max_blocks, n_splits, dtype;
   float scale, lambda, out_scale, eps;
+  const void* gate; int64_t gate_rs;
+  int window, keep_first;
+  float sink;
 } atma_softmax_args;
 
 int atma_softmax_prefill(const atma_softmax_args* args, void* stream);
