@@ -1097,6 +1097,9 @@ def main():
                     help="instead of the default workload: throughput of the Rizurax decoder beside AtmaModel at equal size and its "
                          "kernels beside the like ones; with a name only that kernel's leg (softmax_prefill, softmax_decode, delta_scan, "
                          "delta_step, rows, linear)")
+    ap.add_argument("--zemivik", nargs="?", const="all", default=None, metavar="KERNEL",
+                    help="the same for the Zemivik decoder, beside Rizurax (attention layers only) and AtmaModel (softmax_prefill, "
+                         "softmax_decode, rows, linear)")
     args = ap.parse_args()
     if args.tokens != T_PREFILL:
         T_PREFILL = args.tokens
@@ -1110,14 +1113,16 @@ def main():
     if args.profile:
         profile_case(args.profile)
         return
-    if args.rizurax:
+    if args.rizurax or args.zemivik:
         import bench_decoder
+        import bench_zemivik
+        name, leg, only = ("rizurax", bench_decoder.run, args.rizurax) if args.rizurax else ("zemivik", bench_zemivik.run, args.zemivik)
         torch.cuda.set_device(local_rank)
         sampler = ClockSampler(local_rank)
         sampler.start()
         sampler.mark_begin()
-        res = bench_decoder.run(measured_peaks(), torch.device("cuda", local_rank), None if args.rizurax == "all" else args.rizurax)
-        emit({"bench": "rizurax", "dtype": "bf16", "data": "synthetic", "peaks": measured_peaks(), **res, "clocks": sampler.stop()})
+        res = leg(measured_peaks(), torch.device("cuda", local_rank), None if only == "all" else only)
+        emit({"bench": name, "dtype": "bf16", "data": "synthetic", "peaks": measured_peaks(), **res, "clocks": sampler.stop()})
         return
     args.warmup = max(args.warmup, 3)
 

@@ -35,14 +35,16 @@ def roof(ms, peaks, nbytes=None, flops=None):
 
 
 # ---- whole models ------------------------------------------------------------------------------------------------------
-def rizurax_config(width, layers):
+def rizurax_config(width, layers, attention_every=None):
+    """``attention_every`` n: every n-th layer is attention (default: the third of four)."""
     H = width // 128
     G = max(2, H // 4)
     rot = {"dims": 32, "base": 500000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
     mlp = {"kind": "dense", "ff": 4 * width}
     delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}
     att = {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "diff": 0.4, "scale": 0.125, "rot": rot}}
-    return {"architecture": "Rizurax", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "layers": [att if i % 4 == 2 else delta for i in range(layers)],
+    return {"architecture": "Rizurax", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, 
+            "layers": [att if (i % 4 == 2 if attention_every is None else i % attention_every == 0) else delta for i in range(layers)],
             "embedding": {"bigram": {"buckets": 4093, "mul_prev": 101, "mul_cur": 7}}}
 
 
@@ -74,14 +76,18 @@ def rizurax_weights(cfg, seed, device):
     return w
 
 
-def rizurax_leg(width, layers, prompts, decodes, device):
+def rizurax_leg(width, layers, prompts, decodes, device, attention_every=None):
+    cfg = rizurax_config(width, layers, attention_every)
+    return model_leg(cfg, rizurax_weights(cfg, 5, device), prompts, decodes, device)
+
+
+def model_leg(cfg, weights, prompts, decodes, device):
+    """Prompt and captured decode steps of a configured model through the engine's step builder."""
     from atma_b200.engine import CacheManager, ModelRunner, Sequence, _CapturedStep
-    from atma_b200.rizurax import RizuraxModel
-    cfg = rizurax_config(width, layers)
-    w = rizurax_weights(cfg, 5, device)
-    n_par = sum(t.numel() for t in w.values())
-    model = RizuraxModel(cfg, w, torch.bfloat16, device)
-    del w
+    from atma_b200.registry import model_class
+    n_par = sum(t.numel() for t in weights.values())
+    model = model_class(cfg).from_config(cfg, weights, torch.bfloat16, device)
+    weights.clear()
     out = {"parameters": n_par, "prefill": {}, "decode": {}}
     g = torch.Generator().manual_seed(6)
 
@@ -153,31 +159,32 @@ def atma_leg(width, layers, prompts, decodes, device):
 
 
 # ---- kernels -----------------------------------------------------------------------------------------------------------
+def batch_of(device, n, T, decode=False):
+    """A step of n sequences in a shuffled cache: their whole prompts, or the last of T tokens; and the cache's pages."""
+    from types import SimpleNamespace
+    from atma_b200.engine import CacheManager, ModelRunner, Sequence
+    host = SimpleNamespace(chunked_prefill=True, graph_decode=False, device=device)        # what ModelRunner asks of a model
+    pages = -(-T // BS)
+    cache = CacheManager(n * pages, BS, n, pages)
+    perm = torch.randperm(n * pages, generator=torch.Generator().manual_seed(2)).tolist()
+    cache.free_pages.clear(), cache.free_pages.extend(perm)
+    seqs = [Sequence(i, [0] * T) for i in range(n)]
+    for s in seqs:
+        cache.admit(s), cache.extend(s, T)
+        s.done = T - 1 if decode else 0
+    return ModelRunner(host, cache, None, False).build([(s, 1 if decode else T) for s in seqs], []), n * pages
+
+
 def kernel_legs(peaks, device, only=None):
     """{name: {"rizurax": roofline, "like": [kernel, roofline]}}"""
+    from functools import partial
     import atma_b200 as ab
     from atma_b200 import decoder_ops as ops
-    from atma_b200.engine import Sequence, CacheManager, ModelRunner
     from atma_b200.layer import PackedMaps
     H, G, DK = 8, 2, 128
     g = torch.Generator(device=device).manual_seed(1)
     rnd = lambda *s: torch.randn(*s, device=device, generator=g, dtype=torch.bfloat16)
-    out = {}
-
-    class Host:                                            # what ModelRunner asks of a model
-        chunked_prefill, graph_decode = True, False
-    Host.device = device
-
-    def batch_of(n, T, decode=False):
-        pages = -(-T // BS)
-        cache = CacheManager(n * pages, BS, n, pages)
-        perm = torch.randperm(n * pages, generator=torch.Generator().manual_seed(2)).tolist()
-        cache.free_pages.clear(), cache.free_pages.extend(perm)
-        seqs = [Sequence(i, [0] * T) for i in range(n)]
-        for s in seqs:
-            cache.admit(s), cache.extend(s, T)
-            s.done = T - 1 if decode else 0
-        return ModelRunner(Host, cache, None, False).build([(s, 1 if decode else T) for s in seqs], []), n * pages
+    out, step_of = {}, partial(batch_of, device)
 
     def want(name):
         return only is None or only == name
@@ -186,7 +193,7 @@ def kernel_legs(peaks, device, only=None):
     P["v_null"] = torch.zeros(H, DK, device=device)
     if want("softmax_prefill"):
         T = 32768
-        b, nb = batch_of(1, T)
+        b, nb = step_of(1, T)
         q, kc, vc, o = rnd(T, H, 2, 64), rnd(nb, BS, G, 128), rnd(nb, BS, G, 128), rnd(T, H * 128)
         ms = dev_ms(lambda: ops.softmax_prefill(q, kc, vc, b.prefill, o, scale=0.125, lam=0.3, out_scale=0.6, eps=1e-6), 5)
         fl = 2.0 * (2 * 64 + 2 * 128) * H * T * (T + 1) / 2
@@ -197,7 +204,7 @@ def kernel_legs(peaks, device, only=None):
                                   "like": ["polar_prefill", roof(lk, peaks, flops=4.0 * DK * H * T * (T + 1) / 2)]}
     if want("softmax_decode"):
         B, ctx = 64, 16384
-        b, nb = batch_of(B, ctx, True)
+        b, nb = step_of(B, ctx, True)
         q, kc, vc, o = rnd(B, H, 2, 64), rnd(nb, BS, G, 128), rnd(nb, BS, G, 128), rnd(B, H * 128)
         ms = dev_ms(lambda: ops.softmax_decode(q, kc, vc, b.decode, o, scale=0.125, lam=0.3, out_scale=0.6, eps=1e-6))
         nbytes = B * ctx * G * 256 * 2.0
@@ -207,7 +214,7 @@ def kernel_legs(peaks, device, only=None):
         del kc, vc
     if want("delta_scan"):
         B, T = 8, 16384
-        b, _ = batch_of(B, T)
+        b, _ = step_of(B, T)
         n = B * T
         ch = 2 * H * DK + H * DK
         z = rnd(n, ch + H * DK + 2 * H)
@@ -240,7 +247,7 @@ def kernel_legs(peaks, device, only=None):
         out["head_norm_silu_gate"] = {"shape": f"{n} x {H} x 128", "rizurax": roof(ms_n, peaks, 3.0 * n * H * DK * 2),
                                       "like": ["rms_sigmoid_gate", roof(ln, peaks, 3.0 * tot * H * DK * 2)]}
         del z, parts, q, k, v
-        b2, nb = batch_of(8, tot // 8)
+        b2, nb = step_of(8, tot // 8)
         z = rnd(tot, (H + G) * 128 + G * 128)
         kc2, vc2 = rnd(nb, BS, G, 128), rnd(nb, BS, G, 128)
         table = torch.zeros(tot, 16, 2, device=device)
@@ -252,7 +259,7 @@ def kernel_legs(peaks, device, only=None):
             z = rnd(B, ch + H * DK + 2 * H)
             w = ops.DeltaWeights(*(rnd(H * DK, 4) * 0.4 for _ in range(3)), torch.full((H,), -1.0, device=device), torch.full((H,), -1.0, device=device),
                                  rnd(DK), heads=H, kv_heads=H, dim=DK, vdim=DK, unit_eps=1e-6, q_scale=DK ** -0.5)
-            b, _ = batch_of(B, 64, True)
+            b, _ = step_of(B, 64, True)
             conv = torch.zeros(B, 4, ch, device=device, dtype=torch.bfloat16)
             states = [torch.zeros(B, H, DK, DK, device=device) for _ in range(4)]                # the tables rotate: 4 x B x 0.5 MB
             o = rnd(B, H * DK)
