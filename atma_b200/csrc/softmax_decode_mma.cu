@@ -9,7 +9,9 @@
 // The eight columns are (map, query head) pairs of the group; a K row holds its head's maps side by side, so a column's
 // Q^T is zero outside its own map's channels and one pass over the row serves both maps.  P^T goes back in as the B
 // operand of O^T += V_w^T P^T through a register transpose, as two 16-bit terms (rounded weight and remainder), which
-// keeps the weights at 16 bits of mantissa; both maps share the V fragments.  The reference maximum of a column is raised
+// keeps the weights at 16 bits of mantissa; both maps share the V fragments.  Where four columns are enough for the group
+// the other four hold the same queries again and carry the remainders, so that both terms are one product (COLS = 4).
+// The reference maximum of a column is raised
 // only when a score exceeds it by more than 2^8.
 #include "softmax_attention.cuh"
 #include "mma_sync.cuh"
@@ -25,19 +27,24 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kNegBig = -1e30f;
 constexpr float kRaise = 8.0f;
 
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t a) {
   uint32_t d;
   asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(d) : "r"(a));
   return d;
 }
 
-template <int MAPS, int DIM, int VD, int STAGES>
+template <int MAPS, int DIM, int VD, int STAGES, int COLS>
 __global__ void __launch_bounds__(128, 2)
 softmax_decode_split_kernel(const atma_softmax_args a) {
   constexpr int KD = MAPS * DIM;
   constexpr int KS = KD / 16, MT = VD / 16, CK = KD / 8, CV = VD / 8;
   constexpr int kKBytes = kTileKeys * KD * 2, kVBytes = kTileKeys * VD * 2, kStage = kKBytes + kVBytes;
-  constexpr int GC = 8 / MAPS;                // query heads per CTA
+  constexpr int GC = COLS / MAPS;             // query heads per CTA; a column is a (map, head) pair
   constexpr int OLD = VD + 4;
   extern __shared__ __align__(128) uint8_t sm[];
   const int rep = a.H / a.G, ngrp = (rep + GC - 1) / GC;
@@ -54,7 +61,7 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
   const bool direct = MAPS == 1 && a.n_splits == 1;
   float* stats = a.scratch;                   // [b][h][map][split]{m, l}, then [b][h][map][split][VD]
   float* sacc = a.scratch + (int64_t)a.n_seqs * a.H * MAPS * a.n_splits * 2;
-  auto part = [&](int col) {                  // column = map * GC + head
+  auto part = [&](int col) {                  // column (below COLS) = map * GC + head
     return (((int64_t)b * a.H + h0 + col % GC) * MAPS + col / GC) * a.n_splits + split;
   };
   auto finish = [&](int c, int d, float v) {    // direct form: gate and store channel d of head h0 + c
@@ -85,10 +92,23 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     const int blk = pos / a.block_size;
     return (int64_t)min(max(bt[blk], 0), a.num_blocks - 1) * a.block_size + (pos - blk * a.block_size);
   };
+  // whether the row sees every key of the tile that starts at pos0 (nearly all of them)
+  auto whole = [&](int pos0) { return pos0 + kTileKeys <= n && (pos - pos0 < a.window || pos0 + kTileKeys <= a.keep_first); };
+  constexpr int kKStep = 128 / CK, kVStep = 128 / CV;            // rows between a thread's copies; its 16-byte column is fixed
+  const int64_t k_off = (tid / CK) * krow + tid % CK * 8, v_off = (tid / CV) * vrow + tid % CV * 8;
   auto load_tile = [&](int it) {
     const uint32_t dst = smem_u32(sm + (it % STAGES) * kStage);
     const int pos0 = tiles[tile0 + it] * kTileKeys;
     const int64_t base = tile_in_page ? row_of(pos0) : 0;
+    if (tile_in_page && whole(pos0)) {
+      const uint16_t *kp = K + base * krow + k_off, *vp = V + base * vrow + v_off;
+#pragma unroll
+      for (int j = 0; j < kTileKeys / kKStep; ++j, kp += kKStep * krow) cp_async16(dst + tile_off(tid / CK + j * kKStep, tid % CK * 8, KD), kp);
+#pragma unroll
+      for (int j = 0; j < kTileKeys / kVStep; ++j, vp += kVStep * vrow)
+        cp_async16(dst + kKBytes + tile_off(tid / CV + j * kVStep, tid % CV * 8, VD), vp);
+      return;
+    }
 #pragma unroll
     for (int j = 0; j < kTileKeys * CK / 128; ++j) {
       const int i = tid + j * 128, r = i / CK, ch = i % CK;
@@ -110,10 +130,11 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     cp_async_commit();
   }
 
-  // Q^T as the B operand: column gq = (map gq / GC, head gq % GC), zero outside its map's channels and past the group
+  // Q^T as the B operand: column c = gq mod COLS = (map c / GC, head c % GC), zero outside its map's channels and past the
+  // group
   uint32_t qb[KS][2];
   {
-    const int m = gq / GC, hh = gq % GC;
+    const int m = gq % COLS / GC, hh = gq % GC;
     const bool on = hh < nh;
     const uint16_t* qrow = static_cast<const uint16_t*>(a.q) + ((int64_t)b * a.H + h0 + (on ? hh : 0)) * KD;
 #pragma unroll
@@ -151,12 +172,15 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) S[e] += S2[e];
-    const int key0 = tiles[tile0 + it] * kTileKeys + 16 * warp + gq;
-    const bool ok0 = key0 < n && key_visible(pos, key0, a.window, a.keep_first);
-    const bool ok1 = key0 + 8 < n && key_visible(pos, key0 + 8, a.window, a.keep_first);
+    const int pos0 = tiles[tile0 + it] * kTileKeys;
     float x[4];                               // [key gq][e], [key gq + 8][e]
-    x[0] = ok0 ? S[0] * sc : -INFINITY; x[1] = ok0 ? S[1] * sc : -INFINITY;
-    x[2] = ok1 ? S[2] * sc : -INFINITY; x[3] = ok1 ? S[3] * sc : -INFINITY;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] = S[e] * sc;
+    if (!whole(pos0)) {
+      const int key0 = pos0 + 16 * warp + gq;
+      if (!(key0 < n && key_visible(pos, key0, a.window, a.keep_first))) x[0] = x[1] = -INFINITY;
+      if (!(key0 + 8 < n && key_visible(pos, key0 + 8, a.window, a.keep_first))) x[2] = x[3] = -INFINITY;
+    }
     const float mx[2] = {fmaxf(x[0], x[2]), fmaxf(x[1], x[3])};
     if (__any_sync(0xffffffffu, mx[0] > mref[0] + kRaise || mx[1] > mref[1] + kRaise)) {
 #pragma unroll
@@ -174,13 +198,16 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
       }
     }
     float p[4];
-    p[0] = exp2f(x[0] - mref[0]); p[1] = exp2f(x[1] - mref[1]);
-    p[2] = exp2f(x[2] - mref[0]); p[3] = exp2f(x[3] - mref[1]);
+    p[0] = ex2(x[0] - mref[0]); p[1] = ex2(x[1] - mref[1]);
+    p[2] = ex2(x[2] - mref[0]); p[3] = ex2(x[3] - mref[1]);
     L[0] += p[0] + p[2]; L[1] += p[1] + p[3];
     const uint32_t h01 = pack2<true>(p[0], p[1]), h23 = pack2<true>(p[2], p[3]);
     const float2 f01 = unpack2<true>(h01), f23 = unpack2<true>(h23);
-    const uint32_t pb0 = movmatrix_trans(h01), pb1 = movmatrix_trans(h23);
-    const uint32_t lb0 = movmatrix_trans(pack2<true>(p[0] - f01.x, p[1] - f01.y)), lb1 = movmatrix_trans(pack2<true>(p[2] - f23.x, p[3] - f23.y));
+    const uint32_t l01 = pack2<true>(p[0] - f01.x, p[1] - f01.y), l23 = pack2<true>(p[2] - f23.x, p[3] - f23.y);
+    const bool rem = COLS == 4 && tq >= 2;                       // this thread's columns 2 tq, 2 tq + 1 carry remainders
+    const uint32_t pb0 = movmatrix_trans(rem ? l01 : h01), pb1 = movmatrix_trans(rem ? l23 : h23);
+    uint32_t lb0 = 0u, lb1 = 0u;
+    if constexpr (COLS == 8) { lb0 = movmatrix_trans(l01); lb1 = movmatrix_trans(l23); }
 #pragma unroll
     for (int mt = 0; mt < MT; mt += 4) {
       uint32_t af[4][4];
@@ -188,8 +215,10 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
       for (int q = 0; q < 4; ++q) ldsm_x4_trans(Vsm + tile_off(16 * warp + vk, 16 * (mt + q) + vm, VD), af[q]);
 #pragma unroll
       for (int q = 0; q < 4; ++q) mma16816<true>(O[mt + q], af[q], pb0, pb1);
+      if constexpr (COLS == 8) {
 #pragma unroll
-      for (int q = 0; q < 4; ++q) mma16816<true>(O[mt + q], af[q], lb0, lb1);
+        for (int q = 0; q < 4; ++q) mma16816<true>(O[mt + q], af[q], lb0, lb1);
+      }
     }
   }
   cp_async_wait<0>();
@@ -219,13 +248,21 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
     }
   }
   __syncthreads();
+  auto total = [&](int c, int d) {            // the four warps, both terms
+    float v = 0.f;
+#pragma unroll
+    for (int t = 0; t < 8 / COLS; ++t)
+#pragma unroll
+      for (int w = 0; w < 4; ++w) v += s_o[(8 * w + COLS * t + c) * OLD + d];
+    return v;
+  };
   if (direct) {
     for (int i = tid; i < nh * VD; i += 128) {
       const int c = i / VD, d = i - c * VD;
       const float M = fmaxf(fmaxf(s_m[c], s_m[8 + c]), fmaxf(s_m[16 + c], s_m[24 + c])), s2 = a.sink * kLog2e;
       const float M2 = fmaxf(M, s2), w = exp2f(M - M2);
       const float l = (s_l[c] + s_l[8 + c] + s_l[16 + c] + s_l[24 + c]) * w + exp2f(s2 - M2);
-      const float acc = (s_o[c * OLD + d] + s_o[(8 + c) * OLD + d] + s_o[(16 + c) * OLD + d] + s_o[(24 + c) * OLD + d]) * w;
+      const float acc = total(c, d) * w;
       finish(c, d, l > 0.f ? acc / l : 0.f);
     }
     return;
@@ -233,7 +270,7 @@ softmax_decode_split_kernel(const atma_softmax_args a) {
   for (int i = tid; i < MAPS * GC * VD; i += 128) {
     const int c = i / VD, d = i - c * VD;
     if (c % GC >= nh) continue;
-    sacc[part(c) * VD + d] = s_o[c * OLD + d] + s_o[(8 + c) * OLD + d] + s_o[(16 + c) * OLD + d] + s_o[(24 + c) * OLD + d];
+    sacc[part(c) * VD + d] = total(c, d);
   }
   if (tid < MAPS * GC && tid % GC < nh) {
     const int c = tid;
@@ -289,11 +326,11 @@ int launch(const atma_softmax_args& a, cudaStream_t st) {
   constexpr int kStages = kStage * 3 * 2 <= 224 * 1024 ? 3 : 2;
   constexpr int kMerge = (4 * 8 * (VD + 4) + 64) * 4;
   constexpr int smem = kStages * kStage > kMerge ? kStages * kStage : kMerge;
-  constexpr int GC = 8 / MAPS;
   const int rep = a.H / a.G;
-  auto kern = softmax_decode_split_kernel<MAPS, DIM, VD, kStages>;
+  const int cols = rep * MAPS <= 4 ? 4 : 8, gc = cols / MAPS;
+  auto kern = cols == 4 ? softmax_decode_split_kernel<MAPS, DIM, VD, kStages, 4> : softmax_decode_split_kernel<MAPS, DIM, VD, kStages, 8>;
   ATMA_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  kern<<<dim3(a.n_splits, a.G * ((rep + GC - 1) / GC), a.n_seqs), 128, smem, st>>>(a);
+  kern<<<dim3(a.n_splits, a.G * ((rep + gc - 1) / gc), a.n_seqs), 128, smem, st>>>(a);
   if (MAPS == 2 || a.n_splits > 1) softmax_decode_merge_kernel<MAPS, VD><<<dim3(a.H, a.n_seqs), VD, 0, st>>>(a);
   return launch_status("softmax_decode (mma)");
 }

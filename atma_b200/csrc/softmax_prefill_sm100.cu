@@ -8,7 +8,8 @@
 // runs alone).  A 128-key tile lies inside one page (the page size is a multiple of 128), so the producer turns a key tile
 // into a cache row with one page-table lookup.  Key tiles that no row of the tile sees are left out.
 //
-//   warp 0      TMA producer: the Q tiles once, K and V tiles (stream 0, stream 1, stream 0, ... or shared) through rings
+//   warp 0      TMA producer: the Q tiles once, K and V tiles (stream 0, stream 1, stream 0, ... or shared) through rings,
+//               with one map the output gate's tiles at the end
 //   warp 1      MMA issuer (one lane)
 //   warps 2-3   idle (they complete the first warpgroup, whose registers are handed over)
 //   warps 4-7   softmax of stream 0, one thread per query row (= one TMEM lane), and its epilogue (two maps: half of the
@@ -37,17 +38,24 @@ constexpr float kLazyThreshold = 8.0f;
 
 __device__ int g_softmax_status = 0;
 
-template <int DIM>
+template <int DIM, int VD>
 struct Cfg {
   static constexpr int kMapTile = kBM * DIM * 2;                 // a Q or K tile of one map
   static constexpr int kKSlots = DIM == 64 ? 4 : 3;
+  static constexpr int kVTile = kBN * VD * 2;
+  // one map: the gate tiles of both streams lie over the Q tiles (read once the last scores are there) or, where they are
+  // larger, behind the rings
+  static constexpr bool kGateOverQ = VD <= DIM;
+  static constexpr int kRings = (2 + kKSlots) * kMapTile + kVStages * kVTile;
+  template <int MAPS>
+  static constexpr int bytes() { return kRings + (MAPS == 1 && !kGateOverQ ? 2 * kVTile : 0) + 1024; }
 };
 
 template <int KS>
 struct Barriers {
   uint64_t q_full[2];
   uint64_t k_full[KS], k_empty[KS], v_full[kVStages], v_empty[kVStages];
-  uint64_t s_full[2], p_full[2], o_final[2];
+  uint64_t s_full[2], p_full[2], o_final[2], g_full[2];
 };
 
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
@@ -69,14 +77,17 @@ __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;"
 template <int MAPS, int DIM, int VD>
 __global__ void __launch_bounds__(kThreads, 1)
 softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                             const __grid_constant__ CUtensorMap tmap_v, const atma_softmax_args a) {
-  constexpr int kMapTile = Cfg<DIM>::kMapTile, KS = Cfg<DIM>::kKSlots, kVTile = kBN * VD * 2;
+                             const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_g,
+                             const atma_softmax_args a) {
+  using C = Cfg<DIM, VD>;
+  constexpr int kMapTile = C::kMapTile, KS = C::kKSlots, kVTile = C::kVTile;
   constexpr int kBox = kBM * 128;                                // one 64-channel box of 128 rows
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;                                            // [2 maps]
   uint8_t* sK = sQ + 2 * kMapTile;                               // [KS]
   uint8_t* sV = sK + KS * kMapTile;                              // [kVStages]
+  uint8_t* sG = C::kGateOverQ ? sQ : smem + C::kRings;           // [2 streams], one map
   __shared__ Barriers<KS> bar;
   __shared__ uint32_t s_tmem_base;
   __shared__ int s_abort;
@@ -98,7 +109,7 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
   if (tid == 0) {
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bar.q_full[i], 1); mbar_init(&bar.s_full[i], 1);
-      mbar_init(&bar.p_full[i], 4); mbar_init(&bar.o_final[i], 1);
+      mbar_init(&bar.p_full[i], 4); mbar_init(&bar.o_final[i], 1); mbar_init(&bar.g_full[i], 1);
     }
     for (int i = 0; i < KS; ++i) { mbar_init(&bar.k_full[i], 1); mbar_init(&bar.k_empty[i], 1); }
     for (int i = 0; i < kVStages; ++i) { mbar_init(&bar.v_full[i], 1); mbar_init(&bar.v_empty[i], 1); }
@@ -152,6 +163,16 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
 #pragma unroll
             for (int cb = 0; cb < VD / 64; ++cb)
               tma_load_4d(sV + s * kVTile + cb * kBox, &tmap_v, &bar.v_full[s], (m == 0 ? g0 : g1) * VD + cb * 64, row, 0, 0);
+          }
+        }
+        if (MAPS == 1 && a.gate != nullptr) {
+          const int i = nk * n_kt - 1;                            // once the last K tile is given back nobody reads Q any more
+          ok = ok && (!C::kGateOverQ || mbar_wait(&bar.k_empty[i % KS], (uint32_t)(i / KS) & 1u, abort_flag));
+          for (int m = 0; m < n_streams && ok; ++m) {
+            mbar_arrive_expect_tx(&bar.g_full[m], kVTile);
+#pragma unroll
+            for (int cb = 0; cb < VD / 64; ++cb)
+              tma_load_4d(sG + m * kVTile + cb * kBox, &tmap_g, &bar.g_full[m], (h0 + m) * VD + cb * 64, r_begin + row0, 0, 0);
           }
         }
       }
@@ -305,7 +326,8 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
     // ---- epilogue ----
     if constexpr (MAPS == 1) {                                    // each warpgroup its own head
       if (ok && my_tiles > 0) {
-        ok = __all_sync(0xffffffffu, mbar_wait(&bar.o_final[m], 0, abort_flag));
+        ok = mbar_wait(&bar.o_final[m], 0, abort_flag) && (a.gate == nullptr || mbar_wait(&bar.g_full[m], 0, abort_flag));
+        ok = __all_sync(0xffffffffu, ok);
         tc_fence_after();
       }
       const bool live = ok && my_tiles > 0;
@@ -313,7 +335,7 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
         const float inv = L > 0.f ? 1.0f / L : 0.f;
         const int64_t row = r_begin + row0 + r;
         __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + row * a.out_rs + (int64_t)(h0 + m) * VD;
-        const __nv_bfloat16* gp = static_cast<const __nv_bfloat16*>(a.gate) + row * a.gate_rs + (int64_t)(h0 + m) * VD;
+        const uint8_t* gp = sG + m * kVTile + r * 128;            // this row in the first 64-channel box, 16-byte pieces swizzled
 #pragma unroll 1
         for (int ch = 0; ch < VD; ch += 32) {
           uint32_t u[32];
@@ -329,13 +351,14 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
             float o[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(u[i + e]) * inv;
-            if (a.gate != nullptr) {
-              const uint4 z = *reinterpret_cast<const uint4*>(gp + ch + i);
+            if (a.gate != nullptr && live) {
+              const int c = ch + i;
+              const uint4 z = *reinterpret_cast<const uint4*>(gp + (c >> 6) * kBox + ((((c & 63) >> 3) ^ (r & 7)) << 4));
               const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
-                o[2 * e] *= 1.0f / (1.0f + __expf(-__uint_as_float(zw[e] << 16)));
-                o[2 * e + 1] *= 1.0f / (1.0f + __expf(-__uint_as_float(zw[e] & 0xffff0000u)));
+                o[2 * e] *= __fdividef(1.0f, 1.0f + __expf(-__uint_as_float(zw[e] << 16)));
+                o[2 * e + 1] *= __fdividef(1.0f, 1.0f + __expf(-__uint_as_float(zw[e] & 0xffff0000u)));
               }
             }
             *reinterpret_cast<uint4*>(op + ch + i) = make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]), pack_bf16(o[6], o[7]));
@@ -401,25 +424,27 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
   if (warp == 0) tmem_dealloc(tbase, 512);
 }
 
-int rows_map(CUtensorMap* out, const void* base, int64_t width, int64_t rows) {
+int rows_map(CUtensorMap* out, const void* base, int64_t width, int64_t rows, int64_t row_stride) {
   const uint64_t dims[4] = {(uint64_t)width, (uint64_t)rows, 1, 1};
-  const int64_t strides[3] = {width, width * rows, width * rows};
+  const int64_t strides[3] = {row_stride, row_stride * rows, row_stride * rows};
   const uint32_t box[4] = {64, 128, 1, 1};
   return make_tmap_16bit_4d(out, base, 1, dims, strides, box);
 }
 
 template <int MAPS, int DIM, int VD>
 int launch(const atma_softmax_args& a, cudaStream_t st) {
-  CUtensorMap mq, mk, mv;
-  const int64_t slots = (int64_t)a.num_blocks * a.block_size;
-  int rc = rows_map(&mq, a.q, (int64_t)a.H * MAPS * DIM, a.total_rows);
-  if (rc == ATMA_OK) rc = rows_map(&mk, a.k_cache, (int64_t)a.G * MAPS * DIM, slots);
-  if (rc == ATMA_OK) rc = rows_map(&mv, a.v_cache, (int64_t)a.G * VD, slots);
+  CUtensorMap mq, mk, mv, mg;
+  const int64_t slots = (int64_t)a.num_blocks * a.block_size, wq = (int64_t)a.H * MAPS * DIM, wk = (int64_t)a.G * MAPS * DIM, wv = (int64_t)a.G * VD;
+  int rc = rows_map(&mq, a.q, wq, a.total_rows, wq);
+  if (rc == ATMA_OK) rc = rows_map(&mk, a.k_cache, wk, slots, wk);
+  if (rc == ATMA_OK) rc = rows_map(&mv, a.v_cache, wv, slots, wv);
+  mg = mq;                                                       // not used without a gate
+  if (rc == ATMA_OK && MAPS == 1 && a.gate != nullptr) rc = rows_map(&mg, a.gate, (int64_t)a.H * VD, a.total_rows, a.gate_rs);
   if (rc != ATMA_OK) return rc;
-  constexpr int smem = (2 + Cfg<DIM>::kKSlots) * Cfg<DIM>::kMapTile + kVStages * kBN * VD * 2 + 1024;
+  constexpr int smem = Cfg<DIM, VD>::template bytes<MAPS>();
   auto kern = softmax_prefill_sm100_kernel<MAPS, DIM, VD>;
   ATMA_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  kern<<<dim3(a.n_tiles, MAPS == 2 ? a.H : (a.H + 1) / 2), kThreads, smem, st>>>(mq, mk, mv, a);
+  kern<<<dim3(a.n_tiles, MAPS == 2 ? a.H : (a.H + 1) / 2), kThreads, smem, st>>>(mq, mk, mv, mg, a);
   return launch_status("softmax_prefill (tcgen05)");
 }
 
