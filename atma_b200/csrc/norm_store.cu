@@ -85,7 +85,8 @@ norm_store_kernel(const NormStoreArgs a) {
 template <typename T, int VEC>
 int launch(const NormStoreArgs& a, int rows, cudaStream_t st) {
   const int groups = (a.nq + a.nk + a.nv) / VEC;
-  const int nv = (groups + kThreads - 1) / kThreads;
+  // many rows: two groups per thread, which halves what the sums and roots cost per channel; few rows: the shorter chain
+  const int nv = max((groups + kThreads - 1) / kThreads, rows >= 2048 && groups >= 128 ? 2 : 1);
   ATMA_REQUIRE(nv <= 32, "norm_store: rows of %d channels", groups * VEC);
   const auto threads = [&](int n) { return min(kThreads, ((groups + n - 1) / n + 31) / 32 * 32); };
   if (nv <= 1) norm_store_kernel<T, VEC, 1><<<rows, threads(1), 0, st>>>(a);

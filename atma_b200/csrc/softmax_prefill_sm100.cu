@@ -74,7 +74,8 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
 }
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int MAPS, int DIM, int VD>
+// WIN: a window is set (without one the key tiles are 0, 1, ... and only the last ones need a mask)
+template <int MAPS, int DIM, int VD, bool WIN>
 __global__ void __launch_bounds__(kThreads, 1)
 softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                              const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_g,
@@ -99,9 +100,9 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
   const int seq = a.tile_seq[blockIdx.x], row0 = a.tile_row[blockIdx.x];
   // head and key/value head of each stream; K and V tiles per key tile
   const int h0 = MAPS == 2 ? blockIdx.y : 2 * blockIdx.y, h1 = MAPS == 2 ? h0 : h0 + 1;
-  const int n_streams = h1 < a.H ? 2 : 1;
-  const int g0 = h0 / (a.H / a.G), g1 = min(h1, a.H - 1) / (a.H / a.G);
-  const int nv = g0 == g1 ? 1 : 2, nk = MAPS == 2 ? 2 : nv;
+  const int n_streams = MAPS == 2 || h1 < a.H ? 2 : 1;
+  const int g0 = h0 / (a.H / a.G), g1 = MAPS == 2 ? g0 : min(h1, a.H - 1) / (a.H / a.G);
+  const int nv = MAPS == 2 || g0 == g1 ? 1 : 2, nk = MAPS == 2 ? 2 : nv;
   const int r_begin = a.cu_rows[seq], n_rows = a.cu_rows[seq + 1] - r_begin, start = a.start_pos[seq];
   const KeyTiles tiles(start + row0, start + min(row0 + kBM, n_rows) - 1, a.max_blocks * a.block_size, a.window, a.keep_first, kBN);
   const int n_kt = start < 0 || row0 >= n_rows ? 0 : tiles.n;
@@ -144,7 +145,7 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
         }
         bool ok = true;
         for (int j = 0; j < n_kt && ok; ++j) {
-          const int key0 = tiles[j] * kBN, blk = key0 / a.block_size;
+          const int key0 = (WIN ? tiles[j] : j) * kBN, blk = key0 / a.block_size;
           const int row = min(max(bt[blk], 0), a.num_blocks - 1) * a.block_size + (key0 - blk * a.block_size);
           for (int m = 0; m < nk; ++m) {
             const int i = nk * j + m, s = i % KS;
@@ -253,9 +254,8 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int key0 = tiles[j] * kBN;
-      const int vis = row_ok ? pos + 1 - key0 : 0;                // key columns from win (or below kept) to vis are seen
-      const int win = pos - a.window + 1 - key0, kept = a.keep_first - key0;
+      const int key0 = (WIN ? tiles[j] : j) * kBN;
+      const int vis = row_ok ? pos + 1 - key0 : 0;                // key columns below this one are seen
       uint32_t s[kBN];
 #pragma unroll
       for (int ch = 0; ch < 4; ++ch) tmem_ld32_nowait(tS + ch * 32, &s[ch * 32]);
@@ -267,10 +267,14 @@ softmax_prefill_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
         for (int i = 0; i < kBN; ++i)
           if (i >= vis) s[i] = 0xff800000u;                       // -inf
       }
-      if (win > 0 && kept < kBN) {
+      if constexpr (WIN) {
+        // and of those the ones from win on and the kept ones
+        const int win = pos - a.window + 1 - key0, kept = a.keep_first - key0;
+        if (win > 0 && kept < kBN) {
 #pragma unroll
-        for (int i = 0; i < kBN; ++i)
-          if (i < win && i >= kept) s[i] = 0xff800000u;
+          for (int i = 0; i < kBN; ++i)
+            if (i < win && i >= kept) s[i] = 0xff800000u;
+        }
       }
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
 #pragma unroll
@@ -442,7 +446,9 @@ int launch(const atma_softmax_args& a, cudaStream_t st) {
   if (rc == ATMA_OK && MAPS == 1 && a.gate != nullptr) rc = rows_map(&mg, a.gate, (int64_t)a.H * VD, a.total_rows, a.gate_rs);
   if (rc != ATMA_OK) return rc;
   constexpr int smem = Cfg<DIM, VD>::template bytes<MAPS>();
-  auto kern = softmax_prefill_sm100_kernel<MAPS, DIM, VD>;
+  // a window that no position of this cache outgrows is none
+  const bool win = a.window < (int64_t)a.max_blocks * a.block_size;
+  auto kern = win ? softmax_prefill_sm100_kernel<MAPS, DIM, VD, true> : softmax_prefill_sm100_kernel<MAPS, DIM, VD, false>;
   ATMA_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   kern<<<dim3(a.n_tiles, MAPS == 2 ? a.H : (a.H + 1) / 2), kThreads, smem, st>>>(mq, mk, mv, mg, a);
   return launch_status("softmax_prefill (tcgen05)");
